@@ -57,6 +57,10 @@ struct NbAttnOpts {
   const float* gate;
   int gate_stride;
   int gate_col;
+  int maps;
+  float lambda;
+  float factor;
+  float eps;
   // the first key of the contiguous run that ends at `pos`
   __host__ __device__ __forceinline__ int first_key(int pos) const {
     if (block > 0) return (pos / block) * block;

@@ -359,9 +359,10 @@ attention_decode_mma_kernel(const __nv_bfloat16* q, int q_stride, int q_col,
   if (slot < 0) {   // padding row: zeros, written by split 0
     nb_grid_dependency_wait();
     nb_launch_dependents();
+    const int width = (opt.maps ? group / 2 : group) * HD;
     if (split == 0)
-      for (int i = tid; i < group * HD; i += NT)
-        out[(size_t)r * out_stride + (size_t)kvh * group * HD + i] = nb_from_f32<TOut>(0.0f);
+      for (int i = tid; i < width; i += NT)
+        out[(size_t)r * out_stride + (size_t)kvh * width + i] = nb_from_f32<TOut>(0.0f);
     return;
   }
   const int pos = row_pos[r];
@@ -416,8 +417,14 @@ attention_decode_mma_kernel(const __nv_bfloat16* q, int q_stride, int q_col,
 #pragma unroll
   for (int ks = 0; ks < KS; ++ks) {
     qb[ks][0] = qb[ks][1] = 0u;
-    if (g < group) {
+    if (g < group && opt.maps == 0) {
       const bf16* p = qrow + q_col + (size_t)(kvh * group + g) * HD + ks * 16 + 2 * t;
+      qb[ks][0] = *reinterpret_cast<const uint32_t*>(p);
+      qb[ks][1] = *reinterpret_cast<const uint32_t*>(p + 8);
+    } else if (g < group && (ks * 16 >= HD / 2) == ((g & 1) != 0)) {
+      // a map's query meets its half of the key only: zeros against the other half
+      const bf16* p = qrow + q_col + (size_t)(kvh * group + g) * (HD / 2) + ks * 16 -
+                      (g & 1) * (HD / 2) + 2 * t;
       qb[ks][0] = *reinterpret_cast<const uint32_t*>(p);
       qb[ks][1] = *reinterpret_cast<const uint32_t*>(p + 8);
     }
@@ -581,6 +588,34 @@ attention_decode_mma_kernel(const __nv_bfloat16* q, int q_stride, int q_col,
   }
   __syncthreads();
   // merge the warps -> partial result of this split (maxima in units of log2 e)
+  // A finished number of a head's result: to its place in the output or, with two maps a head, to
+  // shared memory, where `finish_maps` takes the heads' differences.  (A thread overwrites only
+  // what it alone has read.)
+  auto emit = [&](int gh, int c, float v) {
+    if (opt.maps)
+      w_acc[gh * HD + c] = v;
+    else
+      out[(size_t)r * out_stride + (size_t)(kvh * group + gh) * HD + c] = nb_from_f32<TOut>(v);
+  };
+  auto finish_maps = [&]() {
+    if (!opt.maps) return;
+    __syncthreads();
+    for (int hh = warp; hh < group / 2; hh += NW) {
+      const float* a1 = w_acc + (size_t)2 * hh * HD;
+      float u[(HD + 31) / 32], ss = 0.0f;
+#pragma unroll
+      for (int k = 0; k < (HD + 31) / 32; ++k) {
+        const int c = lane + 32 * k;
+        u[k] = c < HD ? a1[c] - opt.lambda * a1[HD + c] : 0.0f;
+        ss = fmaf(u[k], u[k], ss);
+      }
+      const float f = opt.factor / sqrtf(nb_warp_sum(ss) / (float)HD + opt.eps);
+      TOut* dst = out + (size_t)r * out_stride + (size_t)(kvh * (group / 2) + hh) * HD;
+#pragma unroll
+      for (int k = 0; k < (HD + 31) / 32; ++k)
+        if (lane + 32 * k < HD) dst[lane + 32 * k] = nb_from_f32<TOut>(u[k] * f);
+    }
+  };
   unsigned c_remote = 0;    // this split's place in split 0's shared memory
   if constexpr (clustered) {
     asm volatile("barrier.cluster.wait.aligned;\n" ::: "memory");
@@ -604,7 +639,7 @@ attention_decode_mma_kernel(const __nv_bfloat16* q, int q_stride, int q_col,
     if (n_splits == 1) {
       if (sink != nullptr) a *= nb_sink_fix(l, M, sink[head], true);
       a *= opt.gate_of(r, head);
-      out[(size_t)r * out_stride + (size_t)head * HD + c] = nb_from_f32<TOut>(l > 0.0f ? a / l : a);
+      emit(gh, c, l > 0.0f ? a / l : a);
       continue;
     }
     if constexpr (clustered) {
@@ -623,7 +658,10 @@ attention_decode_mma_kernel(const __nv_bfloat16* q, int q_stride, int q_col,
       part_ml[pi * 2 + 1] = l;
     }
   }
-  if (n_splits == 1) return;
+  if (n_splits == 1) {
+    finish_maps();
+    return;
+  }
   if constexpr (clustered) {
     // the stores above are visible to split 0 once every CTA has arrived (release) and split 0
     // has waited (acquire); the other splits wait too, so that none leaves the cluster early
@@ -645,9 +683,9 @@ attention_decode_mma_kernel(const __nv_bfloat16* q, int q_stride, int q_col,
       }
       if (sink != nullptr) a *= nb_sink_fix(l, M, sink[kvh * group + gh], true);
       a *= opt.gate_of(r, kvh * group + gh);
-      out[(size_t)r * out_stride + (size_t)(kvh * group + gh) * HD + c] =
-          nb_from_f32<TOut>(l > 0.0f ? a / l : a);
+      emit(gh, c, l > 0.0f ? a / l : a);
     }
+    finish_maps();
     return;
   }
   __threadfence();
@@ -693,8 +731,9 @@ attention_decode_mma_kernel(const __nv_bfloat16* q, int q_stride, int q_col,
     }
     if (sink != nullptr) a *= nb_sink_fix(l, M, sink[head], true);
     a *= opt.gate_of(r, head);
-    out[(size_t)r * out_stride + (size_t)head * HD + c] = nb_from_f32<TOut>(l > 0.0f ? a / l : a);
+    emit(gh, c, l > 0.0f ? a / l : a);
   }
+  finish_maps();
 }
 
 template <int HD, typename TOut, int MMA_STAGES, int NW>
@@ -934,6 +973,37 @@ NB_EXPORT int nb_attention_decode_capped(const void* q, int dtype, int q_stride,
   return attention_decode(q, dtype, q_stride, q_col, row_slot, row_pos, k_cache, v_cache, block_table,
                           max_pages, page, n_heads, n_kv_heads, head_dim, out, out_dtype, out_stride,
                           scale, softcap, sink, opt, n_rows, n_splits, part_acc, part_ml, counters,
+                          /*append=*/-1, 0, 0, g_cluster_merge.load(), stream);
+}
+
+// Differential heads on the bfloat16 kernel (NbAttnOpts::maps): n_heads of them over n_kv_heads
+// key/value heads of head_dim numbers, a key head's two maps side by side; q: head after head
+// [map 1 | map 2].  The step's keys and values are in the cache already (as above).
+NB_EXPORT int nb_attention_decode_maps_supported(int dtype, int head_dim, int n_heads, int n_kv_heads,
+                                                 int page) {
+  return dtype == NB_BF16 && head_dim % 32 == 0 &&
+         nb_attention_decode_supported(dtype, head_dim, 2 * n_heads, n_kv_heads, page);
+}
+
+NB_EXPORT int nb_attention_decode_maps(const void* q, int q_stride, const int* row_slot,
+                                       const int* row_pos, const void* k_cache, const void* v_cache,
+                                       const int* block_table, int max_pages, int page, int n_heads,
+                                       int n_kv_heads, int head_dim, void* out, int out_stride,
+                                       float scale, int window, float lambda, float factor, float eps,
+                                       int n_rows, int n_splits, float* part_acc, float* part_ml,
+                                       int* counters, cudaStream_t stream) {
+  NB_REQUIRE(nb_attention_decode_maps_supported(NB_BF16, head_dim, n_heads, n_kv_heads, page),
+             NB_ERR_UNSUPPORTED, "attention_decode_maps: unsupported shape (head size %d, %d/%d heads)",
+             head_dim, n_heads, n_kv_heads);
+  NB_REQUIRE(window >= 0, NB_ERR_BAD_ARG, "attention_decode_maps: bad window %d", window);
+  NbAttnOpts opt{window, 0, 0, nullptr, 0, 0};
+  opt.maps = 1;
+  opt.lambda = lambda;
+  opt.factor = factor;
+  opt.eps = eps;
+  return attention_decode(q, NB_BF16, q_stride, 0, row_slot, row_pos, k_cache, v_cache, block_table,
+                          max_pages, page, 2 * n_heads, n_kv_heads, head_dim, out, NB_BF16, out_stride,
+                          scale, 0.0f, nullptr, opt, n_rows, n_splits, part_acc, part_ml, counters,
                           /*append=*/-1, 0, 0, g_cluster_merge.load(), stream);
 }
 

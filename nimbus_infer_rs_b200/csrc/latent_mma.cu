@@ -15,6 +15,10 @@
 // maximum and denominator in scratch memory and `latent_merge_kernel` adds them up.  The sink
 // (a term of the denominator with no key and no value) enters where the row is finished: in
 // the attention kernel without splits, in the merge with.
+//
+// A cached row may hold, behind its `value_dim` numbers that are key and value, numbers that are
+// key only (a rotated part): the score product contracts over the whole row, the value product
+// takes its first numbers.
 #include "mma_common.cuh"
 
 namespace {
@@ -26,14 +30,18 @@ constexpr int PAGE_KEYS = 64;
 constexpr int TILE = 64;       // (token, head) pairs per CTA
 constexpr int THREADS = 128;
 constexpr float LOG2E = 1.4426950408889634f;
+constexpr int MAX_EXTRA = 64;  // key-only numbers behind the values
 
-template <int NT>   // the latent's size rounded up to NT * 16
+// NT: the values' size rounded up to NT * 16; NX: room for key-only numbers behind it, in 16s (the
+// score product runs only the k-steps that hold numbers of the row)
+template <int NT, int NX>
 __global__ void __launch_bounds__(THREADS)
 latent_mma_kernel(const bf16* q, const int* cu_rows, const int* seq_slot, const int* seq_pos0,
-                  const bf16* cache, const int* block_table, int max_pages, int R, int H,
+                  const bf16* cache, const int* block_table, int max_pages, int R, int V, int H,
                   const float* sink, bf16* out, float scale_log2, int window, int n_splits,
                   float* part_o, float* part_ml) {
-  constexpr int RP = NT * 16, LD = RP + 8;
+  constexpr int RP = (NT + NX) * 16, LD = RP + 8;
+  const int k_steps = NX > 0 ? (R + 15) / 16 : NT;
   nb_grid_dependency_wait();
   nb_launch_dependents();
   extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -119,7 +127,8 @@ latent_mma_kernel(const bf16* q, const int* cu_rows, const int* seq_slot, const 
 #pragma unroll
       for (int i = 0; i < 8; ++i) sc[i][0] = sc[i][1] = sc[i][2] = sc[i][3] = 0.0f;
 #pragma unroll
-      for (int kk = 0; kk < NT; ++kk) {
+      for (int kk = 0; kk < NT + NX; ++kk) {
+        if (NX > 0 && kk >= k_steps) break;
         uint32_t a[4];
         ldmatrix_x4(a, Qs + (warp * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * LD + kk * 16 +
                            (lane >> 4) * 8);
@@ -204,11 +213,11 @@ latent_mma_kernel(const bf16* q, const int* cu_rows, const int* seq_slot, const 
     const int tok = r / H, h = r - tok * H;
     const size_t pair = (size_t)(row0 + tok) * H + h;
     if (n_splits > 1) {
-      float* po = part_o + (pair * n_splits + z) * R;
+      float* po = part_o + (pair * n_splits + z) * V;
 #pragma unroll
       for (int i = 0; i < 2 * NT; ++i) {
         const int col = i * 8 + 2 * t4;
-        if (col < R) *reinterpret_cast<float2*>(po + col) = make_float2(o[i][2 * half], o[i][2 * half + 1]);
+        if (col < V) *reinterpret_cast<float2*>(po + col) = make_float2(o[i][2 * half], o[i][2 * half + 1]);
       }
       if (t4 == 0) *reinterpret_cast<float2*>(part_ml + (pair * n_splits + z) * 2) = make_float2(m, l);
     } else {
@@ -220,11 +229,11 @@ latent_mma_kernel(const bf16* q, const int* cu_rows, const int* seq_slot, const 
         l = l * f + exp2_fast(s2 - mf);
       }
       const float inv = l > 0.0f ? f / l : 0.0f;
-      bf16* dst = out + pair * R;
+      bf16* dst = out + pair * V;
 #pragma unroll
       for (int i = 0; i < 2 * NT; ++i) {
         const int col = i * 8 + 2 * t4;
-        if (col < R)
+        if (col < V)
           *reinterpret_cast<uint32_t*>(dst + col) = pack_bf16(o[i][2 * half] * inv, o[i][2 * half + 1] * inv);
       }
     }
@@ -261,22 +270,22 @@ __global__ void latent_merge_kernel(const float* part_o, const float* part_ml, c
   }
 }
 
-template <int NT>
+template <int NT, int NX>
 int launch(const bf16* q, const int* cu_rows, const int* seq_slot, const int* seq_pos0,
-           const bf16* cache, const int* block_table, int max_pages, int R, int H, const float* sink,
+           const bf16* cache, const int* block_table, int max_pages, int R, int V, int H, const float* sink,
            bf16* out, float scale, int window, int n_seqs, int max_q_len, int n_splits,
            float* part_o, float* part_ml, cudaStream_t stream) {
-  constexpr int LD = NT * 16 + 8;
+  constexpr int LD = (NT + NX) * 16 + 8;
   const size_t smem = (size_t)3 * TILE * LD * sizeof(bf16);
   static bool set = false;
   if (!set) {
-    NB_CUDA(cudaFuncSetAttribute(latent_mma_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    NB_CUDA(cudaFuncSetAttribute(latent_mma_kernel<NT, NX>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                  (int)smem));
     set = true;
   }
   const dim3 grid(((size_t)max_q_len * H + TILE - 1) / TILE, n_seqs, n_splits);
-  NB_CUDA(nb_launch(latent_mma_kernel<NT>, grid, dim3(THREADS), smem, stream, q, cu_rows, seq_slot,
-                    seq_pos0, cache, block_table, max_pages, R, H, sink, out, scale * LOG2E, window,
+  NB_CUDA(nb_launch(latent_mma_kernel<NT, NX>, grid, dim3(THREADS), smem, stream, q, cu_rows, seq_slot,
+                    seq_pos0, cache, block_table, max_pages, R, V, H, sink, out, scale * LOG2E, window,
                     n_splits, part_o, part_ml));
   return 0;
 }
@@ -284,46 +293,56 @@ int launch(const bf16* q, const int* cu_rows, const int* seq_slot, const int* se
 }  // namespace
 
 // Whether the tensor-core kernel takes this shape (else the caller uses nb_attention_latent).
-NB_EXPORT int nb_attention_latent_mma_supported(int rank, int page, int n_heads) {
-  return rank % 8 == 0 && rank >= 8 && rank <= 256 && page == PAGE_KEYS && n_heads >= 1;
+NB_EXPORT int nb_attention_latent_mma_supported(int rank, int value_dim, int page, int n_heads) {
+  return rank % 8 == 0 && value_dim % 8 == 0 && value_dim >= 8 && value_dim <= 256 && value_dim <= rank &&
+         rank <= (value_dim + 15) / 16 * 16 + MAX_EXTRA && page == PAGE_KEYS && n_heads >= 1;
 }
 
-// q, out: bf16 [n_rows][n_heads * rank], contiguous; cache: bf16 one plane [n_pages][64][rank];
-// part_o / part_ml: fp32 scratch of n_rows * n_heads * n_splits * rank and ... * 2 numbers
+// q: bf16 [n_rows][n_heads * rank], out: bf16 [n_rows][n_heads * value_dim], contiguous; cache: bf16 one
+// plane [n_pages][64][rank], the first value_dim numbers of a row its values; part_o / part_ml:
+// fp32 scratch of n_rows * n_heads * n_splits * value_dim and ... * 2 numbers
 // (needed when n_splits > 1).  max_q_len: the longest run of rows of one sequence.
 NB_EXPORT int nb_attention_latent_mma(const void* q, const int* cu_rows, const int* seq_slot,
                                       const int* seq_pos0, const int* row_slot, const void* cache,
                                       const int* block_table, int max_pages, int page, int n_heads,
-                                      int rank, const float* sink, void* out, float scale, int window,
+                                      int rank, int value_dim, const float* sink, void* out, float scale,
+                                      int window,
                                       int n_rows, int n_seqs, int max_q_len, int n_splits,
                                       float* part_o, float* part_ml, cudaStream_t stream) {
   if (n_rows == 0 || n_seqs == 0) return 0;
-  NB_REQUIRE(nb_attention_latent_mma_supported(rank, page, n_heads), NB_ERR_UNSUPPORTED,
-             "attention_latent_mma: latent size %d / page %d not supported", rank, page);
+  NB_REQUIRE(nb_attention_latent_mma_supported(rank, value_dim, page, n_heads), NB_ERR_UNSUPPORTED,
+             "attention_latent_mma: rows of %d with %d values / page %d not supported", rank, value_dim,
+             page);
   NB_REQUIRE(n_splits >= 1 && n_splits <= 64 && (n_splits == 1 || (part_o && part_ml)), NB_ERR_BAD_ARG,
              "attention_latent_mma: bad splits %d", n_splits);
   NB_REQUIRE(((uintptr_t)q | (uintptr_t)cache | (uintptr_t)out) % 16 == 0, NB_ERR_BAD_ARG,
              "attention_latent_mma: pointers must be 16-byte aligned");
   NB_REQUIRE(n_seqs <= 65535, NB_ERR_UNSUPPORTED, "attention_latent_mma: too many sequences");
-  const int nt = (rank + 15) / 16;
+  const int nt = (value_dim + 15) / 16;
+  const bool extra = rank > value_dim;
   int rc;
-#define NB_LM(N_)                                                                                  \
-  rc = launch<N_>((const bf16*)q, cu_rows, seq_slot, seq_pos0, (const bf16*)cache, block_table,    \
-                  max_pages, rank, n_heads, sink, (bf16*)out, scale, window, n_seqs, max_q_len,    \
-                  n_splits, part_o, part_ml, stream)
-  if (nt <= 2) NB_LM(2);
-  else if (nt <= 4) NB_LM(4);
-  else if (nt <= 6) NB_LM(6);
-  else if (nt <= 8) NB_LM(8);
-  else if (nt <= 12) NB_LM(12);
-  else NB_LM(16);
+#define NB_LM(N_, X_)                                                                              \
+  rc = launch<N_, X_>((const bf16*)q, cu_rows, seq_slot, seq_pos0, (const bf16*)cache, block_table, \
+                      max_pages, rank, value_dim, n_heads, sink, (bf16*)out, scale, window, n_seqs, \
+                      max_q_len, n_splits, part_o, part_ml, stream)
+#define NB_LM2(N_)                                                                                 \
+  do {                                                                                             \
+    if (extra) NB_LM(N_, MAX_EXTRA / 16); else NB_LM(N_, 0);                                       \
+  } while (0)
+  if (nt <= 2) NB_LM2(2);
+  else if (nt <= 4) NB_LM2(4);
+  else if (nt <= 6) NB_LM2(6);
+  else if (nt <= 8) NB_LM2(8);
+  else if (nt <= 12) NB_LM2(12);
+  else NB_LM2(16);
+#undef NB_LM2
 #undef NB_LM
   if (rc) return rc;
   NB_CHECK_LAUNCH("attention_latent_mma");
   if (n_splits > 1) {
     NB_CUDA(nb_launch(latent_merge_kernel, dim3((unsigned)((size_t)n_rows * n_heads)), dim3(64), 0, stream,
                       (const float*)part_o, (const float*)part_ml, row_slot, sink, (bf16*)out, n_heads,
-                      rank, n_splits));
+                      value_dim, n_splits));
     NB_CHECK_LAUNCH("latent_merge");
   }
   return 0;

@@ -38,13 +38,14 @@ typedef Shape<1, 1, 4, 1, 4> Small;    // 16 places, 128 threads
 // source row is order[place] / row_div, or the place itself) or, with `uniform_rows` > 0, every
 // group has rows 0 .. uniform_rows - 1, reads columns e * x_gcol .. of x and writes columns
 // e * y_gcol .. of y; rows with a negative `row_slot` then give zeros, and with `gate` the
-// result is multiplied by sigmoid(gate[row][gate_col + e]).
+// result is multiplied by sigmoid(gate[row][gate_col + e]), or with gate_each output n's by
+// sigmoid(gate[row][gate_col + e * N + n]).
 template <typename S, bool DUAL, typename TX, typename TY>
 __global__ void __launch_bounds__(S::THREADS)
 moe_mma_kernel(const TX* x, int x_stride, const int* order, int row_div, const int* offsets,
                int n_experts, const bf16* __restrict__ W, const bf16* __restrict__ W2, TY* y,
                int y_stride, int N, int K, int act, float act_param, int uniform_rows, int x_gcol, int y_gcol,
-               const int* row_slot, const float* gate, int gate_stride, int gate_col) {
+               const int* row_slot, const float* gate, int gate_stride, int gate_col, int gate_each) {
   constexpr int BM = S::BM, THREADS = S::THREADS, STAGES = S::STAGES, MI = S::MI, NJ = S::NJ;
   nb_grid_dependency_wait();
   nb_launch_dependents();
@@ -205,8 +206,10 @@ moe_mma_kernel(const TX* x, int x_stride, const int* order, int row_div, const i
       float scale = 1.0f;
       if (uniform_rows > 0) {
         if (a_row[local] < 0) scale = 0.0f;
-        else if (gate != nullptr) scale = nb_sigmoid(gate[(size_t)p * gate_stride + gate_col + e]);
+        else if (gate != nullptr && !gate_each) scale = nb_sigmoid(gate[(size_t)p * gate_stride + gate_col + e]);
       }
+      const float* each = (uniform_rows > 0 && gate != nullptr && gate_each)
+                              ? gate + (size_t)p * gate_stride + gate_col + (size_t)e * N : nullptr;
 #pragma unroll
       for (int nt = 0; nt < 2 * NJ; ++nt) {
 #pragma unroll
@@ -216,6 +219,7 @@ moe_mma_kernel(const TX* x, int x_stride, const int* order, int row_div, const i
           float v = acc[mi][nt][2 * half + c];
           if (DUAL) v = nb_gate_up<true>(v, acc2[mi][nt][2 * half + c], act, act_param);
           else v = nb_apply_act_fast(v, act);
+          if (each != nullptr) v *= nb_sigmoid(each[n]);
           y[(size_t)p * y_stride + n] = nb_from_f32<TY>(scale == 0.0f ? 0.0f : v * scale);
         }
       }
@@ -227,7 +231,7 @@ struct Uniform {      // the per-head form (see the kernel)
   int rows = 0, x_gcol = 0, y_gcol = 0;
   const int* row_slot = nullptr;
   const float* gate = nullptr;
-  int gate_stride = 0, gate_col = 0;
+  int gate_stride = 0, gate_col = 0, gate_each = 0;
 };
 
 // Tiles of a launch: `places` places in `groups` groups (each group rounds up on its own).
@@ -251,7 +255,7 @@ int launch(int tiles, cudaStream_t stream, const TX* x, int x_stride, const int*
   NB_REQUIRE(grid.y <= 65535, NB_ERR_UNSUPPORTED, "grouped product: %d outputs are too many", N);
   NB_CUDA(nb_launch(moe_mma_kernel<S, DUAL, TX, TY>, grid, dim3(S::THREADS), smem, stream, x, x_stride,
                     order, row_div, offsets, n_experts, W, W2, y, y_stride, N, K, act, act_param, u.rows, u.x_gcol,
-                    u.y_gcol, u.row_slot, u.gate, u.gate_stride, u.gate_col));
+                    u.y_gcol, u.row_slot, u.gate, u.gate_stride, u.gate_col, u.gate_each));
   return 0;
 }
 
@@ -304,9 +308,9 @@ NB_EXPORT int nb_head_linear_mma_supported(int x_dtype, int w_dtype, int y_dtype
 }
 
 NB_EXPORT int nb_head_linear_mma(const void* x, int x_dtype, int x_stride, int x_col, const void* W,
-                                 void* y, int y_stride, const float* gate, int gate_stride,
-                                 int gate_col, const int* row_slot, int n_rows, int n_heads, int n_in,
-                                 int n_out, cudaStream_t stream) {
+                                 void* y, int y_stride, int y_hstride, const float* gate,
+                                 int gate_stride, int gate_col, int gate_each, const int* row_slot,
+                                 int n_rows, int n_heads, int n_in, int n_out, cudaStream_t stream) {
   if (n_rows == 0) return 0;
   NB_REQUIRE(nb_head_linear_mma_supported(x_dtype, NB_BF16, NB_BF16, x_stride, x_col, n_in),
              NB_ERR_UNSUPPORTED, "head_linear_mma: shape not supported (in=%d stride=%d col=%d)", n_in,
@@ -314,8 +318,8 @@ NB_EXPORT int nb_head_linear_mma(const void* x, int x_dtype, int x_stride, int x
   NB_REQUIRE((uintptr_t)W % 16 == 0 && (x_dtype == NB_F32 || (uintptr_t)x % 16 == 0), NB_ERR_BAD_ARG,
              "head_linear_mma: pointers must be 16-byte aligned");
   Uniform u;
-  u.rows = n_rows; u.x_gcol = n_in; u.y_gcol = n_out; u.row_slot = row_slot;
-  u.gate = gate; u.gate_stride = gate_stride; u.gate_col = gate_col;
+  u.rows = n_rows; u.x_gcol = n_in; u.y_gcol = y_hstride; u.row_slot = row_slot;
+  u.gate = gate; u.gate_stride = gate_stride; u.gate_col = gate_col; u.gate_each = gate_each;
   int rc;
 #define NB_GO(S_, TX_)                                                                               \
   rc = launch<S_, false, TX_, bf16>(((n_rows + S_::BM - 1) / S_::BM) * n_heads, stream,               \

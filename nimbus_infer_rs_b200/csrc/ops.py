@@ -293,6 +293,49 @@ class CudaBackend:
         self._call("nb_gather_mul", _ptr(g), _ptr(table), dtype_code(table.dtype), _ptr(tokens),
                    _ptr(out), dtype_code(out.dtype), n, d, self._stream())
 
+    def streams(self, x, n_streams, spread, *, write=None, into=None, total=None, read=None, out=None):
+        """One pass over the residual streams of every row.  ``x``: fp32 ``[rows, n_streams * d]``,
+        or with ``spread`` ``[rows, d]``: every stream equals that row.  ``write = (y, ls, mix,
+        gain)``: stream ``t`` becomes ``sum_s mix[s, t] x_s + gain[t] * ls * y``, stored in ``into``
+        (``[rows, n_streams * d]``, may be ``x``; ``None``: not stored) and summed over the streams
+        into ``total`` (``[rows, d]``) where given.  ``read = (coef, gamma, eps)``: ``out`` =
+        rms-norm(``sum_s coef[s] x_s``) ``* gamma`` of the streams as they then are."""
+        _check(x, "x", torch.float32, 2)
+        S = int(n_streams)
+        n, width = x.shape
+        d = width if spread else width // S
+        if not spread and width != S * d:
+            raise KernelError("streams: shapes do not agree")
+        y = ls = mix = gain = coef = gamma = None
+        eps = 0.0
+        if write is not None:
+            y, ls, mix, gain = write
+            _check(y, "y", torch.float32, 2)
+            if y.shape != (n, d) or ls.numel() != d or mix.numel() != S * S or gain.numel() != S:
+                raise KernelError("streams: write-back shapes do not agree")
+        if into is not None:
+            _check(into, "into", torch.float32, 2)
+            if into.shape != (n, S * d) or write is None:
+                raise KernelError("streams: nowhere to store")
+        if total is not None:
+            _check(total, "total", torch.float32, 2)
+            if total.shape != (n, d) or write is None:
+                raise KernelError("streams: the sum's shape does not match")
+        if read is not None:
+            coef, gamma, eps = read
+            _check(out, "out", None, 2)
+            if out.shape != (n, d) or coef.numel() != S or gamma.numel() != d:
+                raise KernelError("streams: read shapes do not agree")
+        self._call("nb_streams", _ptr(x), width, 0 if spread else d, S, _ptr(into), _ptr(y), _ptr(ls),
+                   _ptr(mix), _ptr(gain), _ptr(total), _ptr(coef), _ptr(gamma), float(eps),
+                   _ptr(out if read is not None else None),
+                   dtype_code(out.dtype) if read is not None else 0, n, d, self._stream())
+
+    def softcap_rows(self, x, cap):
+        """``x <- cap * tanh(x / cap)`` in place (fp32)."""
+        _check(x, "x", torch.float32, 2)
+        self._call("nb_softcap_rows", _ptr(x), float(cap), x.numel(), self._stream())
+
     # -- matrix products --------------------------------------------------------------
     def linear(self, x, w, bias, out, act=ACT_NONE, residual=None, norm=None):
         """out = act(norm(x) @ w.T + bias) (+ residual).  x [M,K], w [N,K], out [M,N].
@@ -608,51 +651,84 @@ class CudaBackend:
                    _ptr(kv.block_table), kv.block_table.shape[1], kv.page, kv.head_dim,
                    layout.n_rows, self._stream())
 
-    def head_linear(self, x, x_col, w, out, layout, gate=None, gate_col=0):
+    def head_linear(self, x, x_col, w, out, layout, gate=None, gate_col=0, gate_each=False,
+                    out_stride=None):
         """A linear map per head: ``out[r, h] = w[h] @ x[r, x_col + h*n_in : ...]`` with ``w``
         ``[n_heads, n_out, n_in]``; with ``gate`` (fp32 rows, head ``h``'s logit at column
-        ``gate_col + h``) the head's result is multiplied by the logit's sigmoid."""
+        ``gate_col + h``) the head's result is multiplied by the logit's sigmoid, with
+        ``gate_each`` every number of it by its own (columns ``gate_col + h*n_out ..``).  Head
+        ``h``'s results start at column ``h * out_stride`` (default ``n_out``)."""
         _check(x, "x", None, 2)
         _check(w, "w", None, 3)
         _check(out, "out", None, 2)
         n_heads, n_out, n_in = w.shape
         n = layout.n_rows
+        pitch = n_out if out_stride is None else int(out_stride)
         if x.shape[0] < n or out.shape[0] < n or x.shape[1] < x_col + n_heads * n_in \
-                or out.shape[1] != n_heads * n_out:
+                or pitch < n_out or out.shape[1] != n_heads * pitch:
             raise KernelError("head_linear: shapes do not agree")
         if gate is not None:
             _check(gate, "gate", torch.float32, 2)
-            if gate.shape[0] < n or gate.shape[1] < gate_col + n_heads:
+            if gate.shape[0] < n or gate.shape[1] < gate_col + n_heads * (n_out if gate_each else 1):
                 raise KernelError("head_linear: gate shape does not match")
         if self.use_mma and self.lib.nb_head_linear_mma_supported(
                 dtype_code(x.dtype), dtype_code(w.dtype), dtype_code(out.dtype), x.shape[1], x_col, n_in):
             self._call("nb_head_linear_mma", _ptr(x), dtype_code(x.dtype), x.shape[1], x_col, _ptr(w),
-                       _ptr(out), out.shape[1], _ptr(gate), gate.shape[1] if gate is not None else 0,
-                       gate_col, _ptr(layout.row_slot), n, n_heads, n_in, n_out, self._stream())
+                       _ptr(out), out.shape[1], pitch, _ptr(gate),
+                       gate.shape[1] if gate is not None else 0, gate_col, 1 if gate_each else 0,
+                       _ptr(layout.row_slot), n, n_heads, n_in, n_out, self._stream())
             return
         self._call("nb_head_linear", _ptr(x), dtype_code(x.dtype), x.shape[1], x_col, _ptr(w),
-                   dtype_code(w.dtype), _ptr(out), dtype_code(out.dtype), out.shape[1], _ptr(gate),
-                   gate.shape[1] if gate is not None else 0, gate_col, _ptr(layout.row_slot), n,
-                   n_heads, n_in, n_out, self._stream())
+                   dtype_code(w.dtype), _ptr(out), dtype_code(out.dtype), out.shape[1], pitch,
+                   _ptr(gate), gate.shape[1] if gate is not None else 0, gate_col,
+                   1 if gate_each else 0, _ptr(layout.row_slot), n, n_heads, n_in, n_out,
+                   self._stream())
 
-    def attention_latent(self, q, layout, kv, n_heads, sink, out, scale, window=0):
+    def latent_rope_append(self, src, col, gamma, eps, freq, rot, rot_dims, amplitude, q, q_col, a,
+                           n_heads, layout, kv, write):
+        """The step's cached rows ``[rms(latent) * gamma | rotated key part]`` from columns ``col
+        ..`` of the fp32 rows ``src`` (the latent, then ``rot`` numbers of which the first
+        ``rot_dims`` are turned by position) into the one-plane store ``kv`` (``write``), and the
+        heads' rotated query parts (fp32 ``q``, head ``h`` at ``q_col + h * rot``) into the last
+        ``rot`` numbers of each head of ``a`` (``[rows, n_heads * kv.head_dim]``)."""
+        _check(src, "src", torch.float32, 2)
+        _check(q, "q", torch.float32, 2)
+        _check(a, "a", kv.k.dtype, 2)
+        _check(freq, "freq", torch.float32, 1)
+        n, width = layout.n_rows, kv.head_dim
+        rank = width - rot
+        if kv.n_kv_heads != 1 or rank < 1 or src.shape[0] < n or src.shape[1] < col + width or \
+                q.shape[0] < n or q.shape[1] < q_col + n_heads * rot or a.shape[0] < n or \
+                a.shape[1] != n_heads * width or freq.numel() != rot_dims // 2 or \
+                (gamma is not None and gamma.numel() != rank):
+            raise KernelError("latent_rope_append: shapes do not agree")
+        self._call("nb_latent_rope_append", _ptr(src), src.shape[1], col, _ptr(gamma), float(eps),
+                   _ptr(freq), int(rot), int(rot_dims), float(amplitude), _ptr(q), q.shape[1], q_col,
+                   _ptr(a), dtype_code(a.dtype), n_heads, _ptr(layout.row_slot), _ptr(layout.row_pos),
+                   _ptr(kv.k), dtype_code(kv.k.dtype), _ptr(kv.block_table), kv.block_table.shape[1],
+                   kv.page, rank, 1 if write else 0, n, self._stream())
+
+    def attention_latent(self, q, layout, kv, n_heads, sink, out, scale, window=0, value_dim=None):
         """Causal attention of the packed rows over the cached latents of ``kv`` (one plane: a
         token's latent is its key and its value, for every head).  ``q``: the heads' queries
         mapped into the latent's space, ``[rows, n_heads * rank]``; ``sink``: fp32 ``[n_heads]``
-        logits of a key-less, value-less term of the softmax's denominator, or ``None``."""
+        logits of a key-less, value-less term of the softmax's denominator, or ``None``.
+        ``value_dim``: only the first so many numbers of a cached row are values (the rest is
+        key only), default all."""
         _check(q, "q", None, 2)
         _check(out, "out", None, 2)
         rank = kv.head_dim
+        dv = rank if value_dim is None else int(value_dim)
         n = layout.n_rows
-        if kv.n_kv_heads != 1 or q.shape[1] != n_heads * rank or out.shape[1] != n_heads * rank \
-                or q.shape[0] < n or out.shape[0] < n:
+        if kv.n_kv_heads != 1 or q.shape[1] != n_heads * rank or out.shape[1] != n_heads * dv \
+                or not 1 <= dv <= rank or q.shape[0] < n or out.shape[0] < n:
             raise KernelError("attention_latent: shapes do not agree")
         if sink is not None:
             _check(sink, "sink", torch.float32, 1)
             if sink.numel() != n_heads:
                 raise KernelError("attention_latent: one sink per head")
         if self.use_mma and q.dtype == out.dtype == kv.k.dtype == torch.bfloat16 \
-                and self.lib.nb_attention_latent_mma_supported(rank, kv.page, n_heads):
+                and self.lib.nb_attention_latent_mma_supported(rank, dv, kv.page, n_heads):
             # tensor cores: 64 (token, head) pairs a CTA; the pages of a tile are cut into runs
             # when the launch would leave SMs idle (one-token steps, short prompts)
             ctas = -(-layout.max_q_len * n_heads // 64) * layout.n_seqs
@@ -664,8 +740,8 @@ class CudaBackend:
             if n_splits > 1:
                 need = n * n_heads * n_splits
                 scr = self._latent_scr.get(q.device)
-                if scr is None or scr[1].numel() < need * 2 or scr[0].numel() < need * rank:
-                    scr = (torch.empty(max(need * rank, 1 << 20), dtype=torch.float32, device=q.device),
+                if scr is None or scr[1].numel() < need * 2 or scr[0].numel() < need * dv:
+                    scr = (torch.empty(max(need * dv, 1 << 20), dtype=torch.float32, device=q.device),
                            torch.empty(max(need * 2, 1 << 14), dtype=torch.float32, device=q.device))
                     self._latent_scr[q.device] = scr
                 part_o, part_ml = scr
@@ -674,13 +750,13 @@ class CudaBackend:
                 out[layout.n_tokens:layout.n_rows].zero_()      # padding rows
             self._call("nb_attention_latent_mma", _ptr(q), _ptr(layout.cu_rows), _ptr(layout.seq_slot),
                        _ptr(layout.seq_pos0), _ptr(layout.row_slot), _ptr(kv.k), _ptr(kv.block_table),
-                       kv.block_table.shape[1], kv.page, n_heads, rank, _ptr(sink), _ptr(out), scale,
+                       kv.block_table.shape[1], kv.page, n_heads, rank, dv, _ptr(sink), _ptr(out), scale,
                        window, n, layout.n_seqs, layout.max_q_len, n_splits, _ptr(part_o),
                        _ptr(part_ml), self._stream())
             return
         self._call("nb_attention_latent", _ptr(q), dtype_code(q.dtype), q.shape[1], 0,
                    _ptr(layout.row_slot), _ptr(layout.row_pos), _ptr(kv.k), dtype_code(kv.k.dtype),
-                   _ptr(kv.block_table), kv.block_table.shape[1], kv.page, n_heads, rank,
+                   _ptr(kv.block_table), kv.block_table.shape[1], kv.page, n_heads, rank, dv,
                    _ptr(sink), _ptr(out), dtype_code(out.dtype), out.shape[1], scale, window, n,
                    self._stream())
 
@@ -837,6 +913,55 @@ class CudaBackend:
                    float(scale), float(softcap or 0.0), int(window), int(keep_first), int(chunk),
                    _ptr(gate), gate.shape[1] if gate is not None else 0, int(gate_col), n,
                    self._stream())
+
+    def attention_differential(self, q, layout, k_store, v_store, n_heads, out, scale, window, lam,
+                               factor, eps):
+        """Differential attention of the packed rows: ``n_heads`` query heads of two maps side by
+        side (``q``: ``[rows, n_heads * 2 d]``) over key heads of two maps (``k_store``, heads of
+        ``2 d``) and values of ``v_store`` (the same store of two planes, or one of its own).  Each
+        map is a softmax attention over the last ``window`` tokens (0: all earlier ones) of the
+        same values; ``o = A_1 - lam * A_2``, then ``o / sqrt(mean(o^2) + eps) * factor`` per head."""
+        _check(q, "q", None, 2)
+        _check(out, "out", None, 2)
+        n, d2, dv = layout.n_rows, k_store.head_dim, v_store.head_dim
+        G, page, code = k_store.n_kv_heads, k_store.page, dtype_code(q.dtype)
+        shared = v_store is k_store
+        if d2 % 2 or q.shape != (n, n_heads * d2) or out.shape != (n, n_heads * dv) or \
+                G != v_store.n_kv_heads or n_heads % G or q.dtype != k_store.k.dtype or \
+                k_store.k.dtype != v_store.k.dtype or (shared and k_store.v is None):
+            raise KernelError("attention_differential: shapes do not agree")
+        v_plane = k_store.v if shared else v_store.k
+        if layout.is_decode and shared and out.dtype == torch.bfloat16 and self.use_mma and \
+                self.lib.nb_attention_decode_maps_supported(code, d2, n_heads, G, page):
+            # one-token steps: the split decode kernel with two maps a head
+            pages = max(1, -(-layout.max_kv_len // page))
+            if window > 0:
+                pages = min(pages, (window + page - 1) // page + 1)
+            n_splits = self._decode_splits(n * G, pages, k_store, q.dtype)
+            acc, ml, counters = self._decode_scratch(q.device, n, 2 * n_heads, G, d2, n_splits)
+            self._call("nb_attention_decode_maps", _ptr(q), q.shape[1], _ptr(layout.row_slot),
+                       _ptr(layout.row_pos), _ptr(k_store.k), _ptr(v_plane), _ptr(k_store.block_table),
+                       k_store.block_table.shape[1], page, n_heads, G, d2, _ptr(out), out.shape[1],
+                       float(scale), int(window), float(lam), float(factor), float(eps), n, n_splits,
+                       _ptr(acc), _ptr(ml), _ptr(counters), self._stream())
+            return
+        if self.use_mma and out.dtype == torch.bfloat16 and \
+                self.lib.nb_attention_differential_mma_supported(code, d2 // 2, dv, page, q.shape[1]):
+            if layout.n_rows > layout.n_tokens:
+                out[layout.n_tokens:layout.n_rows].zero_()      # padding rows
+            self._call("nb_attention_differential_mma", _ptr(q), q.shape[1], _ptr(layout.cu_rows),
+                       _ptr(layout.seq_slot), _ptr(layout.seq_pos0), _ptr(k_store.k),
+                       _ptr(k_store.block_table), k_store.block_table.shape[1], _ptr(v_plane),
+                       _ptr(v_store.block_table), v_store.block_table.shape[1], page, n_heads, G,
+                       d2 // 2, dv, _ptr(out), float(scale), int(window), float(lam), float(factor),
+                       float(eps), layout.n_seqs, layout.max_q_len, self._stream())
+            return
+        self._call("nb_attention_differential", _ptr(q), code, _ptr(layout.row_slot),
+                   _ptr(layout.row_pos), _ptr(k_store.k), _ptr(k_store.block_table),
+                   k_store.block_table.shape[1], _ptr(v_plane), _ptr(v_store.block_table),
+                   v_store.block_table.shape[1], dtype_code(k_store.k.dtype), page, n_heads, G, d2 // 2,
+                   dv, _ptr(out), dtype_code(out.dtype), float(scale), int(window), float(lam),
+                   float(factor), float(eps), n, self._stream())
 
     def pool_blocks(self, layout, kv, blocks, pool):
         """For every row that completes a block of ``pool`` tokens: the means of the block's keys

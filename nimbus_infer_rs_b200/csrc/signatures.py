@@ -82,14 +82,22 @@ SIGNATURES = {
     "nb_layernorm": "pppppiiifp",
     "nb_rmsnorm": "piipppiiifp",
     "nb_latent_append": "piipfpppipiiiip",
-    "nb_head_linear": "piiipipiipiipiiiip",
-    "nb_attention_latent": "piiipppipiiiippiifiip",
-    "nb_attention_latent_mma_supported": "iii",
-    "nb_attention_latent_mma": "pppppppiiiippfiiiiippp",
+    "nb_latent_rope_append": "piipfpiifpiipiipppipiiiiip",
+    "nb_head_linear": "piiipipiiipiiipiiiip",
+    "nb_attention_latent": "piiipppipiiiiippiifiip",
+    "nb_attention_latent_mma_supported": "iiii",
+    "nb_attention_latent_mma": "pppppppiiiiippfiiiiippp",
+    "nb_streams": "piiippppppppfpiiip",
+    "nb_softcap_rows": "pflp",
+    "nb_attention_differential": "pippppippiiiiiiipififffip",
+    "nb_attention_differential_mma_supported": "iiiii",
+    "nb_attention_differential_mma": "pipppppippiiiiiipfifffiip",
+    "nb_attention_decode_maps_supported": "iiiii",
+    "nb_attention_decode_maps": "pipppppiiiiipififffiipppp",
     "nb_moe_gemm_mma_supported": "iiii",
     "nb_moe_gemm_mma": "pipipiipppiiiiifp",
     "nb_head_linear_mma_supported": "iiiiii",
-    "nb_head_linear_mma": "piiippipiipiiiip",
+    "nb_head_linear_mma": "piiippiipiiipiiiip",
     "nb_moe_gemm_tc_set_wait_budget": "l",
     "nb_moe_gemm_tc_supported": "iiiiii",
     "nb_moe_gather": "pipipipiip",

@@ -29,3 +29,9 @@ class StepContext:
     # the stream and leaves them in ``normed``)
     next_norm: Any = None
     normed: Any = None
+    # ... and that entry's arrangement itself (None after the last entry)
+    next_block: Any = None
+    # residual streams: the single row they all equal until the first of them is written, and
+    # (set by the last entry's arrangement) their sum at the end
+    streams_from: Any = None
+    streams_sum: Any = None

@@ -50,7 +50,7 @@ class Layer:
 
     def parts(self):
         """The layer's parts that exist, by the name their parameters are listed under."""
-        named = {"norm_mixer": self.norm_mixer, "mixer": self.mixer,
+        named = {"block": self.block, "norm_mixer": self.norm_mixer, "mixer": self.mixer,
                  "norm_ffn": self.norm_ffn, "ffn": self.ffn,
                  "post_norm_mixer": self.post_norm_mixer, "post_norm_ffn": self.post_norm_ffn,
                  "side": self.side}
@@ -74,7 +74,7 @@ class Model:
         self.stream_input = build_part("stream", spec.stream_input) \
             if spec.stream_input is not None else None
         self.stream_input_before = frozenset(spec.stream_input_before)
-        self.head = LMHead(spec.vocab_size, spec.width, spec.tie_head)
+        self.head = LMHead(spec.vocab_size, spec.width, spec.tie_head, spec.logit_softcap)
         self.run_order = spec.run_order()
         self.params: dict[str, torch.Tensor | None] = {}
 
@@ -109,7 +109,7 @@ class Model:
         if self.stream_input is not None:
             parts.append(self.stream_input)
         for l in self.layers:
-            parts += [l.block, *l.parts().values()]
+            parts += l.parts().values()
         return all(getattr(p, "graph_safe", False) for p in parts)
 
     def n_params(self) -> int:
@@ -138,6 +138,11 @@ class Model:
             # the layers add into the stream in place: the embedding's output is kept apart
             x = torch.empty_like(x0)
             ctx.ops.cast_cols(x0, x, 0)
+        if self.spec.streams > 1:
+            # the streams all equal the embedding's output until a sublayer writes them
+            ctx.streams_from = x0
+            x = torch.empty((x0.shape[0], self.spec.streams * self.spec.width), device=x0.device,
+                            dtype=torch.float32)
         for entry, li in enumerate(self.run_order):
             layer = self.layers[li]
             if entry in self.stream_input_before:
@@ -147,13 +152,16 @@ class Model:
             ctx.kv_extra = ctx.cache.layer_kv_extra(entry)
             # an arrangement whose last pass over the stream can also norm it for the entry that
             # runs next is told that entry's first norm
-            ctx.next_norm = None
+            ctx.next_norm = ctx.next_block = None
             if entry + 1 < len(self.run_order) and entry + 1 not in self.stream_input_before:
                 nxt = self.layers[self.run_order[entry + 1]]
-                if getattr(nxt.block, "takes_handed_norm", False):
+                ctx.next_block = nxt.block
+                if getattr(nxt.block, "takes_handed_norm", False) and type(nxt.block) is type(layer.block):
                     ctx.next_norm = nxt.norm_mixer
             layer.block.forward(ctx, x, layer)
-        ctx.next_norm = ctx.normed = None
+        ctx.next_norm = ctx.normed = ctx.next_block = None
+        if self.spec.streams > 1:
+            x, ctx.streams_sum = ctx.streams_sum, None
         return x
 
     def storage_requests(self):

@@ -11,7 +11,10 @@ an arrangement in which both sublayers read one norm has no second norm (``norm_
 ``stream_input`` with ``stream_input_before``: a part of the ``stream`` family (one set of
 parameters) that transforms the stream right before each of the named schedule entries, from
 the stream and the embedding's output.  ``logit_scale`` multiplies the logits.  ``embedding``: a
-part of the ``embedding`` family in place of the plain token table.
+part of the ``embedding`` family in place of the plain token table.  ``streams`` > 1: the residual
+is that many streams of the model's width side by side (all equal to the embedding's output at
+first, their sum goes to the final norm), which only the ``hyper_connections`` arrangement runs
+on.  ``logit_softcap`` > 0: logits ``z`` become ``logit_softcap * tanh(z / logit_softcap)``.
 """
 from __future__ import annotations
 
@@ -48,6 +51,8 @@ class ModelSpec:
     schedule: tuple[int, ...] | None = None
     embedding_scale: float = 1.0      # multiplies the token embedding (not the tied head)
     logit_scale: float = 1.0          # multiplies the logits
+    logit_softcap: float = 0.0        # bounds the logits (0: no bound)
+    streams: int = 1                  # residual streams side by side
     # another way from tokens to the stream than the token table (``embedding`` family); its
     # arguments must include ``vocab_size`` and ``width``
     embedding: PartSpec | None = None
@@ -63,12 +68,18 @@ class ModelSpec:
 
     def validate(self) -> None:
         n_entries = len(self.run_order())
+        if self.streams < 1 or (self.streams > 1 and self.stream_input is not None):
+            raise ValueError("a stream input acts on one residual stream")
         if self.stream_input_before and self.stream_input is None:
             raise ValueError("stream_input_before names entries, but there is no stream_input")
         for e in self.stream_input_before:
             if not 0 <= e < n_entries:
                 raise ValueError(f"stream_input_before names entry {e} of {n_entries}")
         for i, l in enumerate(self.layers):
+            if l.block.args.get("streams", 1) != self.streams:
+                raise ValueError(f"layer {i}: arrangement {l.block.kind!r} runs on "
+                                 f"{l.block.args.get('streams', 1)} residual streams, the model has "
+                                 f"{self.streams}")
             if l.cache_from is not None:
                 if not 0 <= l.cache_from < len(self.layers) or l.cache_from == i:
                     raise ValueError(f"layer {i}: cache_from={l.cache_from} is not another layer")

@@ -4,3 +4,4 @@ from . import runesun  # noqa: F401
 from . import rizitar  # noqa: F401
 from . import pinozen  # noqa: F401
 from . import lulizen  # noqa: F401
+from . import bumulix  # noqa: F401

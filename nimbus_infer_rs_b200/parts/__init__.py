@@ -9,12 +9,13 @@ from .attention import CausalSelfAttention
 from .latent_attention import LatentAttention
 from .feed_forward import DenseMLP, GatedMLP
 from .routed_experts import RoutedExperts
-from .block import ParallelBlock, PreNormBlock, SandwichBlock
+from .block import HyperConnectionsBlock, ParallelBlock, PreNormBlock, SandwichBlock
 from .pooled_attention import PooledWindowAttention
 from .delta_rule import DeltaRule
 from .token_side import GatedTokenInput
 from .capped_attention import CappedAttention
 from .masked_attention import MaskedAttention
+from .differential_attention import DifferentialAttention
 from .selective_scan import SelectiveScan
 from .linear_attention import DecayedLinearAttention
 from .mixer_pair import NormedPair

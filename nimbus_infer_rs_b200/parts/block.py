@@ -3,7 +3,8 @@ from __future__ import annotations
 
 import torch
 
-from .base import Block, register_part
+from .base import VECTOR, Block, ParamSpec, register_part
+from .norm import RMSNorm
 
 
 @register_part("block", "pre_norm")
@@ -97,3 +98,112 @@ class SandwichBlock(Block):
         ctx.normed, xr = last.add_into(ctx, y, x, then=then, rounded=wants_rounded)
         if side is not None:
             side.forward(ctx, x, xr if wants_rounded else x)
+
+
+@register_part("block", "hyper_connections")
+class HyperConnectionsBlock(Block):
+    """Several residual streams: a sublayer reads a weighted sum of them, and its result is written
+    back to all while they are mixed with one another.  For sublayer ``q`` (1 mixer, 2
+    feed-forward, which may be absent) of a layer
+
+        ``u = sum_s in_q[s] x_s``;  ``y = ls_q * sublayer(norm(u))``;
+        ``x_t <- sum_s mix_q[s, t] x_s + residual_mult * out_q[t] * y``   (all from the old streams)
+
+    ``ls_q`` scales the result number by number (``layer_scale=False``: not).  ``streams=1`` with
+    ``connections=False`` is the ordinary residual with a layer scale and a multiplier.
+
+    ``x`` is fp32 ``[rows, streams * width]``, stream after stream.  One pass over a row writes a
+    sublayer's result back and hands out what reads the streams next: the normed rows of the
+    layer's feed-forward, those of the next layer's mixer (left in ``ctx.normed``), or at the end
+    of the model the sum of the streams (``ctx.streams_sum``).  The first write-back of a step
+    reads the embedding's single row (``ctx.streams_from``), which all streams equal until then."""
+    graph_safe = True
+    takes_handed_norm = True
+
+    def __init__(self, width: int, streams: int = 1, residual_mult: float = 1.0,
+                 layer_scale: bool = True, connections: bool = True, ffn: bool = True):
+        self.width, self.streams = int(width), int(streams)
+        self.residual_mult = float(residual_mult)
+        self.layer_scale, self.connections = bool(layer_scale), bool(connections)
+        if self.streams > 1 and not self.connections:
+            raise ValueError("several streams need their connections")
+        self.sublayers = (1, 2) if ffn else (1,)
+        for q in (1, 2):
+            for n in ("in", "out", "mix", "scale", "gain"):
+                setattr(self, f"{n}{q}", None)
+
+    def param_specs(self):
+        S, specs = self.streams, {}
+        for q in self.sublayers:
+            if self.connections:
+                specs.update({f"in{q}": ParamSpec((S,), VECTOR), f"out{q}": ParamSpec((S,), VECTOR),
+                              f"mix{q}": ParamSpec((S, S), VECTOR)})
+            if self.layer_scale:
+                specs[f"scale{q}"] = ParamSpec((self.width,), VECTOR)
+        return specs
+
+    def bind(self, params, runtime) -> None:
+        super().bind(params, runtime)
+        one = torch.ones(1, dtype=torch.float32, device=runtime.device)
+        for q in self.sublayers:
+            if not self.connections:
+                setattr(self, f"in{q}", one)
+                setattr(self, f"out{q}", one)
+                setattr(self, f"mix{q}", one.view(1, 1))
+            if not self.layer_scale:
+                setattr(self, f"scale{q}", torch.ones(self.width, dtype=torch.float32,
+                                                      device=runtime.device))
+            out = getattr(self, f"out{q}")
+            setattr(self, f"gain{q}", None if out is None else (out * self.residual_mult).contiguous())
+
+    def _source(self, ctx, x):
+        """The tensor the streams are read from, and whether it is their common single row."""
+        if ctx.streams_from is not None:
+            return ctx.streams_from, True
+        return x, False
+
+    def _read(self, q: int, norm):
+        if not isinstance(norm, RMSNorm):
+            raise ValueError("residual streams are read through root-mean-square norms")
+        return getattr(self, f"in{q}"), norm.weight, norm.eps
+
+    def _write_back(self, ctx, x, y, q: int, read):
+        """Sublayer ``q``'s result into the streams; returns the rows of the next read."""
+        src, spread = self._source(ctx, x)
+        last = read is None and self.streams > 1 and ctx.next_block is None
+        out = torch.empty_like(y, dtype=ctx.rt.act_dtype) if read is not None else None
+        total = torch.empty_like(y) if last else None
+        ctx.ops.streams(src, self.streams, spread,
+                        write=(y, getattr(self, f"scale{q}"), getattr(self, f"mix{q}"),
+                               getattr(self, f"gain{q}")),
+                        into=None if last else x, total=total, read=read, out=out)
+        ctx.streams_from = None
+        if last:
+            ctx.streams_sum = total
+        return out
+
+    @staticmethod
+    def _run(part, ctx, h, y):
+        if getattr(part, "can_overwrite", False):
+            part.forward(ctx, h, y, accumulate=False)
+        else:
+            part.forward(ctx, h, y.zero_())
+
+    def forward(self, ctx, x, layer) -> None:
+        n, dev = x.shape[0], x.device
+        h, ctx.normed = ctx.normed, None
+        if h is None:
+            src, spread = self._source(ctx, x)
+            h = torch.empty((n, self.width), device=dev, dtype=ctx.rt.act_dtype)
+            ctx.ops.streams(src, self.streams, spread, read=self._read(1, layer.norm_mixer), out=h)
+        y = torch.empty((n, self.width), device=dev, dtype=torch.float32)
+        self._run(layer.mixer, ctx, h, y)
+        nxt = ctx.next_block
+        hand_over = nxt._read(1, ctx.next_norm) if isinstance(nxt, HyperConnectionsBlock) else None
+        if layer.ffn is None:
+            ctx.normed = self._write_back(ctx, x, y, 1, hand_over)
+            return
+        h = self._write_back(ctx, x, y, 1, self._read(2, layer.norm_ffn))
+        y = torch.empty((n, self.width), device=dev, dtype=torch.float32)
+        self._run(layer.ffn, ctx, h, y)
+        ctx.normed = self._write_back(ctx, x, y, 2, hand_over)

@@ -74,15 +74,17 @@ class HashedPairEmbedding(TokenEmbedding):
 
 class LMHead(Part):
     """``logits = h @ W.T`` without bias, fp32 result; ``W`` is the token embedding table when
-    tied (src/model.rs:317-325)."""
+    tied (src/model.rs:317-325).  ``softcap`` > 0 replaces a logit ``z`` by ``softcap * tanh(z /
+    softcap)``."""
     graph_safe = True
     family = "head"
     kind = "lm_head"
 
-    def __init__(self, vocab_size: int, width: int, tied: bool):
+    def __init__(self, vocab_size: int, width: int, tied: bool, softcap: float = 0.0):
         self.vocab_size = int(vocab_size)
         self.width = int(width)
         self.tied = bool(tied)
+        self.softcap = float(softcap or 0.0)
         self.weight = None
 
     def param_specs(self):
@@ -100,4 +102,6 @@ class LMHead(Part):
             h, norm = h.x, h.args
         logits = torch.empty((h.shape[0], self.vocab_size), device=h.device, dtype=torch.float32)
         ctx.ops.linear(h, self.weight, None, logits, 0, None, norm)
+        if self.softcap > 0.0:
+            ctx.ops.softcap_rows(logits, self.softcap)
         return logits

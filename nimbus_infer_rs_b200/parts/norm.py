@@ -58,12 +58,14 @@ class RMSNorm(Norm):
     defers: one launch gives the rows to every reader."""
     graph_safe = True
 
-    def __init__(self, width: int, eps: float, gain: float = 1.0):
+    def __init__(self, width: int, eps: float, gain: float = 1.0, zero_centred: bool = False):
         """``gain``: a constant that multiplies the result (a model that scales its logits does
-        so through its last norm); folded into the weight when it is bound."""
+        so through its last norm); ``zero_centred``: the stored weight ``w`` means ``1 + w``.  Both
+        are folded into the weight (fp32) when it is bound."""
         self.width = int(width)
         self.eps = float(eps)
         self.gain = float(gain)
+        self.zero_centred = bool(zero_centred)
         self.weight = None
 
     def param_specs(self):
@@ -71,6 +73,8 @@ class RMSNorm(Norm):
 
     def bind(self, params, runtime) -> None:
         super().bind(params, runtime)
+        if self.zero_centred and self.weight is not None:
+            self.weight = (self.weight + 1.0).contiguous()
         if self.gain != 1.0 and self.weight is not None:
             self.weight = (self.weight * self.gain).contiguous()
 

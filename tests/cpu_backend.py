@@ -203,6 +203,48 @@ class CpuBackend:
                     o = o * torch.sigmoid(gate[r, gate_col + h])
                 out[r, h * dv:(h + 1) * dv] = o.to(out.dtype)
 
+    def attention_differential(self, q, layout, k_store, v_store, n_heads, out, scale, window, lam,
+                               factor, eps):
+        d2, dv, G = k_store.head_dim, v_store.head_dim, k_store.n_kv_heads
+        group, d = n_heads // G, d2 // 2
+        for r in range(layout.n_rows):
+            slot = int(layout.row_slot[r])
+            if slot < 0:
+                out[r].zero_()
+                continue
+            pos = int(layout.row_pos[r])
+            idx = torch.arange(max(0, pos + 1 - window) if window > 0 else 0, pos + 1)
+            at, inside = (idx // k_store.page).long(), (idx % k_store.page).long()
+            k = k_store.k[k_store.block_table[slot, at].long(), :, inside].float()     # [n, G, 2 d]
+            v = (k_store.v if v_store is k_store else v_store.k)[
+                v_store.block_table[slot, at].long(), :, inside].float()               # [n, G, dv]
+            for h in range(n_heads):
+                qh = q[r, h * d2:(h + 1) * d2].float()
+                a = []
+                for m in (slice(0, d), slice(d, d2)):
+                    a.append(torch.softmax(k[:, h // group, m] @ qh[m] * scale, 0) @ v[:, h // group])
+                u = a[0] - lam * a[1]
+                u = u / torch.sqrt((u * u).mean() + eps) * factor
+                out[r, h * dv:(h + 1) * dv] = u.to(out.dtype)
+
+    def streams(self, x, n_streams, spread, *, write=None, into=None, total=None, read=None, out=None):
+        n = x.shape[0]
+        xs = x[:, None, :].repeat(1, n_streams, 1) if spread else x.view(n, n_streams, -1).clone()
+        if write is not None:
+            y, ls, mix, gain = write
+            xs = torch.einsum("nsd,st->ntd", xs, mix) + gain[None, :, None] * (ls * y)[:, None, :]
+            if into is not None:
+                into.copy_(xs.reshape(n, -1))
+            if total is not None:
+                total.copy_(xs.sum(1))
+        if read is not None:
+            coef, gamma, eps = read
+            u = torch.einsum("nsd,s->nd", xs, coef)
+            out.copy_((u / torch.sqrt((u * u).mean(-1, keepdim=True) + eps) * gamma).to(out.dtype))
+
+    def softcap_rows(self, x, cap):
+        x.copy_(cap * torch.tanh(x / cap))
+
     def pool_blocks(self, layout, kv, blocks, pool):
         for r in range(layout.n_rows):
             slot = int(layout.row_slot[r])
@@ -441,18 +483,48 @@ class CpuBackend:
             page = int(kv.block_table[slot, pos // kv.page])
             kv.k[page, 0, pos % kv.page, :] = v.to(kv.k.dtype)
 
-    def head_linear(self, x, x_col, w, out, layout, gate=None, gate_col=0):
+    def latent_rope_append(self, src, col, gamma, eps, freq, rot, rot_dims, amplitude, q, q_col, a,
+                           n_heads, layout, kv, write):
+        width = kv.head_dim
+        rank, half = width - rot, rot_dims // 2
+
+        def turn(x, pos):
+            ang = float(pos) * freq
+            c, s = torch.cos(ang) * amplitude, torch.sin(ang) * amplitude
+            u, v = x[..., :half], x[..., half:rot_dims]
+            return torch.cat([u * c - v * s, v * c + u * s, x[..., rot_dims:]], -1)
+
+        heads = a.view(-1, n_heads, width)
+        for r in range(layout.n_rows):
+            slot = int(layout.row_slot[r])
+            if slot < 0:
+                heads[r, :, rank:] = 0
+                continue
+            pos = int(layout.row_pos[r])
+            qr = q[r, q_col:q_col + n_heads * rot].view(n_heads, rot)
+            heads[r, :, rank:] = turn(qr, pos).to(a.dtype)
+            if write:
+                c = src[r, col:col + rank]
+                c = c / torch.sqrt((c * c).mean() + eps) * (gamma if gamma is not None else 1.0)
+                row = torch.cat([c, turn(src[r, col + rank:col + width], pos)])
+                page = int(kv.block_table[slot, pos // kv.page])
+                kv.k[page, 0, pos % kv.page, :] = row.to(kv.k.dtype)
+
+    def head_linear(self, x, x_col, w, out, layout, gate=None, gate_col=0, gate_each=False,
+                    out_stride=None):
         n = layout.n_rows
         n_heads, n_out, n_in = w.shape
         xs = x[:n, x_col:x_col + n_heads * n_in].float().view(n, n_heads, n_in)
         y = torch.einsum("rhi,hoi->rho", xs, w.float())
         if gate is not None:
-            y = y * torch.sigmoid(gate[:n, gate_col:gate_col + n_heads])[:, :, None]
+            k = n_out if gate_each else 1
+            y = y * torch.sigmoid(gate[:n, gate_col:gate_col + n_heads * k]).view(n, n_heads, k)
         y = torch.where((layout.row_slot[:n] >= 0)[:, None, None], y, torch.zeros_like(y))
-        out[:n].copy_(y.reshape(n, n_heads * n_out).to(out.dtype))
+        out[:n].view(n, n_heads, out_stride or n_out)[:, :, :n_out] = y.to(out.dtype)
 
-    def attention_latent(self, q, layout, kv, n_heads, sink, out, scale, window=0):
+    def attention_latent(self, q, layout, kv, n_heads, sink, out, scale, window=0, value_dim=None):
         rank = kv.head_dim
+        dv = rank if value_dim is None else value_dim
         for r in range(layout.n_rows):
             slot = int(layout.row_slot[r])
             if slot < 0:
@@ -472,7 +544,7 @@ class CpuBackend:
             den = e.sum(-1)
             if sink is not None:
                 den = den + torch.exp(sink - m)
-            out[r] = ((e / den[:, None]) @ c).reshape(-1).to(out.dtype)
+            out[r] = ((e / den[:, None]) @ c[:, :dv]).reshape(-1).to(out.dtype)
 
     def moe_route(self, logits, col, n_experts, top, renormalize, layout, idx, weight):
         n = layout.n_rows
