@@ -21,7 +21,7 @@ events around exactly K captured steps), ``e2e`` = the same through the Python e
 
 ``python bench.py --designs`` is another measurement with a line of its own (the default
 workload and its line stay as they are): with ``--design`` one of the other designs (Runesun,
-Rizitar, Pinozen, Lulizen) beside GPT-2 or the closest design; by default the Runesun design (latent attention, routed experts)
+Rizitar, Pinozen, Lulizen, Bumulix) beside GPT-2 or the closest design; by default the Runesun design (latent attention, routed experts)
 beside GPT-2 at equal layer sizes (presets ``runesun-2k`` / ``gpt2-2k`` and ``runesun-1k`` /
 ``gpt2-1k``, random weights): decode steps at batch 8 and 64 and a 2 x 1024-token prefill, and
 per kind of kernel the time inside a plainly launched step with its bytes, flops and fraction of
@@ -296,7 +296,11 @@ DESIGN_PAIRS = {"runesun": (("runesun-2k", "gpt2-2k"), ("runesun-1k", "gpt2-1k")
                 "pinozen": (("pinozen-2k", "rizitar-2k"), ("pinozen-1k", "rizitar-1k")),
                 # beside the closest design of the library: sublayers between two norms, attention
                 # with normed and rotated queries and keys over a window, routed experts
-                "lulizen": (("lulizen-2k", "rizitar-2k"), ("lulizen-1k", "rizitar-1k"))}
+                "lulizen": (("lulizen-2k", "rizitar-2k"), ("lulizen-1k", "rizitar-1k")),
+                # beside the two closest designs: Lulizen's masked attention over shared key heads
+                # and Runesun's attention over a latent
+                "bumulix": (("bumulix-2k", "lulizen-2k", "runesun-2k"),
+                            ("bumulix-1k", "lulizen-1k", "runesun-1k"))}
 
 
 class OpTimer:
@@ -310,7 +314,8 @@ class OpTimer:
              "attention_pooled", "delta_rule", "conv_rope_append", "conv_act", "attention_capped",
              "selective_scan", "linear_attention", "rmsnorm_gated", "rms_pair_add", "glu_rows",
              "cast_cols", "embed_hashed", "ln_add", "qkv_norm_rope_append",
-             "attention_masked", "moe_route_sigmoid")
+             "attention_masked", "moe_route_sigmoid", "attention_differential",
+             "latent_rope_append", "streams", "softcap_rows")
 
     def __init__(self, ops):
         import torch
@@ -371,9 +376,11 @@ class OpTimer:
                 per_key, planes = kv.n_kv_heads * kv.head_dim, 2
                 width = heads * kv.head_dim
             else:
-                q, lay, kv, heads = a[0], a[1], a[2], a[3]
-                per_key, planes = kv.head_dim, 1
-                width = heads * kv.head_dim
+                q, lay, kv, heads, out = a[0], a[1], a[2], a[3], a[5]
+                keys = sum(p + n for p, n in zip(lay.seq_pos0_host, lay.seq_lens))
+                pairs = sum(n * p + n * (n + 1) // 2 for p, n in zip(lay.seq_pos0_host, lay.seq_lens))
+                return keys * kv.head_dim * kv.k.element_size() + nb(q, out), \
+                    2 * pairs * (q.shape[1] + out.shape[1])
             elt = kv.k.element_size()
             keys = sum(p + n for p, n in zip(lay.seq_pos0_host, lay.seq_lens))
             pairs = sum(n * p + n * (n + 1) // 2 for p, n in zip(lay.seq_pos0_host, lay.seq_lens))
@@ -420,6 +427,26 @@ class OpTimer:
                        for p, n in zip(lay.seq_pos0_host, lay.seq_lens))
             return keys * ks.n_kv_heads * (ks.head_dim + vs.head_dim) * elt + nb(q, out), \
                 2 * pairs * heads * (ks.head_dim + vs.head_dim)
+        if kind == "attention_differential":
+            q, lay, ks, vs, heads, out, window = a[0], a[1], a[2], a[3], a[4], a[5], a[7]
+
+            def first(i):
+                return max(0, i + 1 - window) if window else 0
+            pairs = sum(i + 1 - first(i) for p, n in zip(lay.seq_pos0_host, lay.seq_lens)
+                        for i in range(p, p + n))
+            keys = sum(p + n - first(p) for p, n in zip(lay.seq_pos0_host, lay.seq_lens))
+            # two maps of half a key each, both over the whole values
+            return keys * ks.n_kv_heads * (ks.head_dim + vs.head_dim) * ks.k.element_size() + nb(q, out), \
+                2 * pairs * heads * (ks.head_dim + 2 * vs.head_dim)
+        if kind == "latent_rope_append":
+            rot, q, heads, lay, kv = a[5], a[8], a[11], a[12], a[13]
+            return lay.n_tokens * ((kv.head_dim + heads * rot) * (4 + kv.k.element_size())), 0
+        if kind == "streams":
+            x, S, spread = a[0], a[1], a[2]
+            y = kw["write"][0] if kw.get("write") else None
+            return nb(x, y, kw.get("into"), kw.get("total"), kw.get("out") if kw.get("read") else None), 0
+        if kind == "softcap_rows":
+            return 2 * nb(a[0]), 0
         if kind == "act_rows":
             return 4 * a[4].numel() + nb(a[4]), 0
         if kind == "gather_mul":

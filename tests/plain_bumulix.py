@@ -176,7 +176,9 @@ def owner(cfg, i):
 
 def sublayer(xs, W, p, q, f, cfg):
     """Sublayer q (1: mixer, 2: feed-forward) of the layer with prefix p around the function f."""
-    eps, m = cfg["norm"]["eps"], cfg["residual_mult"]
+    eps, m = cfg["norm"]["eps"], cfg.get("residual_mult", 1.0)
+    if cfg.get("streams") is None:                     # an ordinary residual
+        return xs + m * W[f"{p}ls{q}"] * f(zero_centred_norm(xs[0], W[f"{p}norm{q}"], eps))
     hc = f"{p}hc{q}."
     y = f(zero_centred_norm(read_streams(xs, W[hc + "in"]), W[f"{p}norm{q}"], eps)) * W[f"{p}ls{q}"]
     return write_streams(xs, W[hc + "mix"], W[hc + "out"], y, m)
@@ -195,7 +197,7 @@ def hidden_states(tokens, W, cfg, dtype=torch.float64):
     """The sum of the streams after every layer run, [runs, T, D]."""
     W = widened(W, dtype)
     x = W["embed"][torch.tensor(list(tokens))]
-    xs = torch.stack([x] * cfg["streams"])
+    xs = torch.stack([x] * cfg.get("streams", 1))
     out = []
     for i in range(len(cfg["layers"])):
         xs = layer_forward(xs, W, cfg, i)
