@@ -196,6 +196,8 @@ moe_mma_kernel(const TX* x, int x_stride, const int* order, int row_div, const i
   cp_async_wait<0>();
   if (!warp_has_rows) return;
   const int g = lane >> 2, t4 = lane & 3;
+  // neighbouring 16-bit results leave together when every row starts on a 4-byte boundary
+  const bool pairs = sizeof(TY) == 2 && y_stride % 2 == 0 && (reinterpret_cast<uintptr_t>(y) & 3) == 0;
 #pragma unroll
   for (int mi = 0; mi < MI; ++mi) {
 #pragma unroll
@@ -212,15 +214,26 @@ moe_mma_kernel(const TX* x, int x_stride, const int* order, int row_div, const i
                               ? gate + (size_t)p * gate_stride + gate_col + (size_t)e * N : nullptr;
 #pragma unroll
       for (int nt = 0; nt < 2 * NJ; ++nt) {
+        const int n = n0 + col_w + nt * 8 + 2 * t4;
+        float v[2];
 #pragma unroll
         for (int c = 0; c < 2; ++c) {
-          const int n = n0 + col_w + nt * 8 + 2 * t4 + c;
-          if (n >= N) continue;
-          float v = acc[mi][nt][2 * half + c];
-          if (DUAL) v = nb_gate_up<true>(v, acc2[mi][nt][2 * half + c], act, act_param);
-          else v = nb_apply_act_fast(v, act);
-          if (each != nullptr) v *= nb_sigmoid(each[n]);
-          y[(size_t)p * y_stride + n] = nb_from_f32<TY>(scale == 0.0f ? 0.0f : v * scale);
+          v[c] = acc[mi][nt][2 * half + c];
+          if (DUAL) v[c] = nb_gate_up<true>(v[c], acc2[mi][nt][2 * half + c], act, act_param);
+          else v[c] = nb_apply_act_fast(v[c], act);
+        }
+        if (each != nullptr) {
+          if (n < N) v[0] *= nb_sigmoid(each[n]);
+          if (n + 1 < N) v[1] *= nb_sigmoid(each[n + 1]);
+        }
+        v[0] = scale == 0.0f ? 0.0f : v[0] * scale;
+        v[1] = scale == 0.0f ? 0.0f : v[1] * scale;
+        TY* dst = y + (size_t)p * y_stride + n;
+        if (sizeof(TY) == 2 && pairs && n + 1 < N) {
+          *reinterpret_cast<uint32_t*>(dst) = pack_bf16(v[0], v[1]);
+        } else {
+          if (n < N) dst[0] = nb_from_f32<TY>(v[0]);
+          if (n + 1 < N) dst[1] = nb_from_f32<TY>(v[1]);
         }
       }
     }

@@ -419,7 +419,7 @@ class CudaBackend:
     # A kernel whose bounded wait on a barrier ran out says so in a word of pinned host memory
     # (one per kernel family); its results are not valid.
     _ERROR_WORDS = {0: "gemm_tcgen05", 1: "attention_prefill_tc", 2: "wait_probe", 3: "gemm_stream",
-                    4: "gemm_tc_rows"}
+                    4: "gemm_tc_rows", 5: "attention_differential_tc"}
 
     def raise_device_errors(self) -> None:
         """Raise if a kernel that has finished reported a timed-out wait.  Reads host memory
@@ -442,7 +442,7 @@ class CudaBackend:
         cycles = 4_000_000_000 if cycles is None else int(cycles)
         for fn in ("nb_gemm_tcgen05_set_wait_budget", "nb_attention_prefill_tc_set_wait_budget",
                    "nb_gemm_stream_set_wait_budget", "nb_gemm_tc_rows_set_wait_budget",
-                   "nb_moe_gemm_tc_set_wait_budget"):
+                   "nb_moe_gemm_tc_set_wait_budget", "nb_attention_differential_tc_set_wait_budget"):
             rc = getattr(self.lib, fn)(cycles)
             if rc != 0:
                 raise KernelError(f"{fn} failed ({rc}): "
@@ -944,6 +944,18 @@ class CudaBackend:
                        k_store.block_table.shape[1], page, n_heads, G, d2, _ptr(out), out.shape[1],
                        float(scale), int(window), float(lam), float(factor), float(eps), n, n_splits,
                        _ptr(acc), _ptr(ml), _ptr(counters), self._stream())
+            return
+        if not layout.is_decode and shared and out.dtype == torch.bfloat16 and self.use_tcgen05 and \
+                scale > 0 and self.lib.nb_attention_differential_tc_supported(code, d2, n_heads, G, page):
+            # prompts, maps of 32 or 64 numbers: tcgen05 tiles of 128 rows
+            if layout.n_rows > layout.n_tokens:
+                out[layout.n_tokens:layout.n_rows].zero_()      # padding rows
+            self._call("nb_attention_differential_tc", _ptr(q), q.shape[0], _ptr(layout.cu_rows),
+                       _ptr(layout.seq_slot), _ptr(layout.seq_pos0), _ptr(k_store.k), _ptr(v_plane),
+                       k_store.k.shape[0], _ptr(k_store.block_table), k_store.block_table.shape[1],
+                       page, n_heads, G, d2, _ptr(out), out.shape[1], float(scale), int(window),
+                       float(lam), float(factor), float(eps), layout.n_seqs, layout.max_q_len,
+                       self._stream())
             return
         if self.use_mma and out.dtype == torch.bfloat16 and \
                 self.lib.nb_attention_differential_mma_supported(code, d2 // 2, dv, page, q.shape[1]):

@@ -45,7 +45,7 @@ def model(vocab, width, layers, streams=None, mult=None, cap=None, eps=1e-5):
     return cfg
 
 
-_A1 = latent(3, 10, 6, 14, 20, 18, 0.3, 500.0, (4.0, 64, 8.0, 0.5))
+_A1 = latent(3, 14, 10, 12, 20, 18, 0.3, 500.0, (4.0, 64, 8.0, 0.5))
 # A: odd sizes; values of another size than two keys (two stores); a window shorter than a page; a
 #    layer without feed-forward; layers that run with another's tensors, beside each other and apart
 # B: multiples of 16 (the tensor-core kernels): values of twice a map's size over shared key heads,

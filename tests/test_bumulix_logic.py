@@ -52,7 +52,7 @@ def test_config_is_read_and_recognised(models):
     a = typed.layers[0].mixer
     assert (a.heads, a.kv_heads, a.dim, a.vdim, a.scale, a.diff, a.mask_size) == (4, 2, 12, 20, 0.3, 0.4, 9)
     b = typed.layers[1].mixer
-    assert (b.heads, b.dim, b.rot_dim, b.vdim, b.kv_rank, b.q_rank) == (3, 10, 6, 14, 20, 18)
+    assert (b.heads, b.dim, b.rot_dim, b.vdim, b.kv_rank, b.q_rank) == (3, 14, 10, 12, 20, 18)
     assert b.rot.base == 500.0 and b.rot.scaling() == {"factor": 4.0, "original": 64.0, "fast": 8.0, "slow": 0.5}
     assert typed.layers[2].weights_of == 1 and typed.owner(2) == 1 and typed.layers[3].mlp is None
     for n in NAMES:
@@ -74,7 +74,7 @@ def test_config_is_read_and_recognised(models):
 def test_config_errors_name_every_bad_key():
     bad = copy.deepcopy(BM.CONFIGS["A"])
     bad["layers"][0]["mixer"]["heads"] = 3                     # no multiple of kv_heads
-    bad["layers"][1]["mixer"]["rot"]["dims"] = 8               # more than rot_dim
+    bad["layers"][1]["mixer"]["rot"]["dims"] = 12              # more than rot_dim
     del bad["layers"][1]["mixer"]["rot"]["scaling"]["fast"]
     bad["layers"][2]["mixer"] = {"heads": 3}
     bad["layers"][3]["type"] = "windowed"
@@ -210,7 +210,7 @@ def test_storage_per_run(models, cpu_backend):
     assert sorted(kv) == [0, 1, 2, 3, 4] and st == {}
     assert kv[0] == kv[4] == KVRequest(2, 24, 9, planes=1)
     assert extra[(0, 0)] == extra[(4, 0)] == KVRequest(2, 20, 9, planes=1)
-    assert kv[1] == kv[2] == KVRequest(1, 26, 0, planes=1)
+    assert kv[1] == kv[2] == KVRequest(1, 30, 0, planes=1)
     assert kv[3] == KVRequest(1, 48, 40, planes=1)
     assert e.cache.layer_kv(1).k.data_ptr() != e.cache.layer_kv(2).k.data_ptr()
     two = _engine(models, "B").model.storage_requests()[0]
@@ -241,14 +241,9 @@ def test_greedy_generation_through_the_engines_loop(models, cpu_backend):
     out = e.generate(prompts, SamplingParams(max_new_tokens=8, temperature=0.0), max_batch=3)
     for p, got in zip(prompts, out):
         assert len(got) == 8
-        ctx = list(p)
-        for tok in got:
-            logits = PB.logits(ctx, P, cfg)[-1]
-            want = int(torch.argmax(logits))
-            if tok != want:
-                assert float(logits[want] - logits[tok]) <= 1e-4 * float(logits.abs().max())
-                break
-            ctx.append(tok)
+        ref = PB.logits(list(p) + got[:-1], P, cfg)[len(p) - 1:]
+        for z, tok in zip(ref, got):      # only a near tie may differ
+            assert float(z.max() - z[tok]) <= 1e-4 * float(z.abs().max())
     assert e.cache.slots.n_free == 3
 
 

@@ -19,7 +19,7 @@ NAMES = list(BM.CONFIGS)
 # root-mean-square difference over the vocabulary relative to the spread of the logits (a head's
 # difference of two maps is brought to unit size, so rounding of a small difference counts in
 # full); the mechanisms alone are held to 2e-5 and 2e-2 in test_gpu_bumulix_kernels.py.
-TOL = {"float32": 1e-4, "bfloat16": 4e-2}
+TOL = {"float32": 1e-4, "bfloat16": 6e-2}
 
 
 def assert_close(got, ref, dtype, what=""):
@@ -42,6 +42,15 @@ def _cases(names):
     """Every configuration in both precisions, except C in bfloat16: its norms over one or two
     numbers are sign functions, which rounding flips."""
     return [(n, d) for n in names for d in DTYPES if not (n == "C" and d == "bfloat16")]
+
+
+@pytest.fixture(scope="module", autouse=True)
+def _few_threads():
+    """The plain implementation's matrices are small: many threads only wait for one another."""
+    n = torch.get_num_threads()
+    torch.set_num_threads(2)
+    yield
+    torch.set_num_threads(n)
 
 
 @pytest.fixture(scope="module")
@@ -192,14 +201,9 @@ def test_greedy_generation_through_the_engines_loop(models):
     out = e.generate(prompts, SamplingParams(max_new_tokens=12, temperature=0.0), max_batch=3)
     for p, got in zip(prompts, out):
         assert len(got) == 12
-        ctx = list(p)
-        for tok in got:
-            logits = PB.logits(ctx, P, cfg)[-1]
-            want = int(torch.argmax(logits))
-            if tok != want:        # only a near tie may differ, and the comparison ends there
-                assert float(logits[want] - logits[tok]) <= 2 * TOL["float32"] * float(logits.abs().max())
-                break
-            ctx.append(tok)
+        ref = PB.logits(list(p) + got[:-1], P, cfg)[len(p) - 1:]
+        for z, tok in zip(ref, got):      # only a near tie may differ
+            assert float(z.max() - z[tok]) <= 2 * TOL["float32"] * float(z.abs().max())
     assert e.cache.slots.n_free == 3
 
 

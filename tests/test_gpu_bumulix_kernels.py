@@ -21,6 +21,15 @@ TOL = {"float32": 2e-5, "bfloat16": 2e-2}
 DTYPES = ["float32", "bfloat16"]
 
 
+@pytest.fixture(scope="module", autouse=True)
+def _few_threads():
+    """The plain implementation's matrices are small: many threads only wait for one another."""
+    n = torch.get_num_threads()
+    torch.set_num_threads(2)
+    yield
+    torch.set_num_threads(n)
+
+
 @pytest.fixture(scope="module")
 def ops():
     return ops_mod.backend()
@@ -176,6 +185,31 @@ def test_attention_whole_in_portions_and_token_by_token(ops, dtype, shape):
     for pieces in ((T,), (2, 61, 1, 2, 64, 3, 142), (202,) + (1,) * 73):
         got = _attention(ops, dtype, q, k, v, pieces, fill=float("nan"), **kw)
         _close(got, ref, TOL[dtype], f"shape {shape} in pieces {pieces[:3]}")
+    if dtype == "bfloat16" and dv == 2 * d and d in (32, 64):
+        # the same heads on the mma.sync prompt kernel, which takes them when tcgen05 is off
+        ops.use_tcgen05 = False
+        try:
+            got = _attention(ops, dtype, q, k, v, (2, 61, 1, 2, 64, 3, 142), fill=float("nan"), **kw)
+        finally:
+            ops.use_tcgen05 = True
+        _close(got, ref, TOL[dtype], f"shape {shape} without tcgen05")
+
+
+@pytest.mark.parametrize("d", [32, 64])
+def test_scores_that_grow_along_the_keys(ops, d):
+    """Every key's score is far above those before it, in one map rising and in the other falling:
+    the exponents' reference moves at every turn, or never, and a result that is not rescaled with
+    it is far off."""
+    T, H, G = 700, 2, 1
+    q, k, v = _rnd(T, H, 2, d, seed=1, s=0.1), _rnd(T, G, 2, d, seed=2, s=0.1), _rnd(T, G, 2 * d, seed=3)
+    q[:, :, :, 0] = 1.0
+    ramp = torch.linspace(0.0, 60.0, T).bfloat16().float()[:, None]
+    k[:, :, 0, 0], k[:, :, 1, 0] = ramp, ramp.flip(0)
+    for window in (0, 300):
+        kw = dict(window=window, scale=1.0, lam=0.5, diff=0.3, eps=1e-5)
+        ref = _plain(q, k, v, **kw)
+        for pieces in ((T,), (130, 570)):
+            _close(_attention(ops, "bfloat16", q, k, v, pieces, **kw), ref, TOL["bfloat16"], f"{window} {pieces}")
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
