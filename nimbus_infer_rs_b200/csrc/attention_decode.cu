@@ -311,7 +311,8 @@ __device__ __forceinline__ uint32_t pack2_bf16(float lo, float hi) {
 // shared memory, two rounds of tensor-core instructions with the softmax between them), so
 // when the CTAs of a launch fit on the GPU with four pages each, eight warps take two pages
 // at a time; a large batch has four warps and two pages per CTA, for more CTAs per SM.
-template <int HD, typename TOut, int MMA_STAGES, bool CLUSTERED, int NW>
+// MAPS: differential heads (NbAttnOpts::maps).
+template <int HD, typename TOut, int MMA_STAGES, bool CLUSTERED, int NW, bool MAPS>
 __global__ void __launch_bounds__(NW * 32)
 attention_decode_mma_kernel(const __nv_bfloat16* q, int q_stride, int q_col,
                             const int* row_slot, const int* row_pos,
@@ -359,7 +360,7 @@ attention_decode_mma_kernel(const __nv_bfloat16* q, int q_stride, int q_col,
   if (slot < 0) {   // padding row: zeros, written by split 0
     nb_grid_dependency_wait();
     nb_launch_dependents();
-    const int width = (opt.maps ? group / 2 : group) * HD;
+    const int width = (MAPS ? group / 2 : group) * HD;
     if (split == 0)
       for (int i = tid; i < width; i += NT)
         out[(size_t)r * out_stride + (size_t)kvh * width + i] = nb_from_f32<TOut>(0.0f);
@@ -417,11 +418,11 @@ attention_decode_mma_kernel(const __nv_bfloat16* q, int q_stride, int q_col,
 #pragma unroll
   for (int ks = 0; ks < KS; ++ks) {
     qb[ks][0] = qb[ks][1] = 0u;
-    if (g < group && opt.maps == 0) {
+    if (!MAPS && g < group) {
       const bf16* p = qrow + q_col + (size_t)(kvh * group + g) * HD + ks * 16 + 2 * t;
       qb[ks][0] = *reinterpret_cast<const uint32_t*>(p);
       qb[ks][1] = *reinterpret_cast<const uint32_t*>(p + 8);
-    } else if (g < group && (ks * 16 >= HD / 2) == ((g & 1) != 0)) {
+    } else if (MAPS && g < group && (ks * 16 >= HD / 2) == ((g & 1) != 0)) {
       // a map's query meets its half of the key only: zeros against the other half
       const bf16* p = qrow + q_col + (size_t)(kvh * group + g) * (HD / 2) + ks * 16 -
                       (g & 1) * (HD / 2) + 2 * t;
@@ -592,13 +593,13 @@ attention_decode_mma_kernel(const __nv_bfloat16* q, int q_stride, int q_col,
   // shared memory, where `finish_maps` takes the heads' differences.  (A thread overwrites only
   // what it alone has read.)
   auto emit = [&](int gh, int c, float v) {
-    if (opt.maps)
+    if constexpr (MAPS)
       w_acc[gh * HD + c] = v;
     else
       out[(size_t)r * out_stride + (size_t)(kvh * group + gh) * HD + c] = nb_from_f32<TOut>(v);
   };
   auto finish_maps = [&]() {
-    if (!opt.maps) return;
+    if constexpr (!MAPS) return;
     __syncthreads();
     for (int hh = warp; hh < group / 2; hh += NW) {
       const float* a1 = w_acc + (size_t)2 * hh * HD;
@@ -736,7 +737,7 @@ attention_decode_mma_kernel(const __nv_bfloat16* q, int q_stride, int q_col,
   finish_maps();
 }
 
-template <int HD, typename TOut, int MMA_STAGES, int NW>
+template <int HD, typename TOut, int MMA_STAGES, int NW, bool MAPS>
 int launch_mma_s(const void* q, int q_stride, int q_col, const int* row_slot, const int* row_pos,
                  const NbPagedKV& kv, int group, void* out, int out_stride, float scale, float softcap, const float* sink, NbAttnOpts opt,
                  int n_rows, int n_splits, float* part_acc, float* part_ml, int* counters, int append,
@@ -746,7 +747,7 @@ int launch_mma_s(const void* q, int q_stride, int q_col, const int* row_slot, co
   const size_t most = tiles + (size_t)MAX_CLUSTER * 8 * (HD + 2) * sizeof(float);
   dim3 grid(n_splits, kv.n_kv_heads, n_rows);
   if (clustered) {
-    auto kern = attention_decode_mma_kernel<HD, TOut, MMA_STAGES, true, NW>;
+    auto kern = attention_decode_mma_kernel<HD, TOut, MMA_STAGES, true, NW, MAPS>;
     static bool configured = false;   // per instantiation
     if (most > 48 * 1024 && !configured) {
       NB_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)most));
@@ -759,7 +760,7 @@ int launch_mma_s(const void* q, int q_stride, int q_col, const int* row_slot, co
                                counters, append, k_col, v_col));
     return 0;
   }
-  auto kern = attention_decode_mma_kernel<HD, TOut, MMA_STAGES, false, NW>;
+  auto kern = attention_decode_mma_kernel<HD, TOut, MMA_STAGES, false, NW, MAPS>;
   static bool configured = false;   // per instantiation
   if (tiles > 48 * 1024 && !configured) {
     NB_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)tiles));
@@ -771,7 +772,7 @@ int launch_mma_s(const void* q, int q_stride, int q_col, const int* row_slot, co
   return 0;
 }
 
-template <int HD, typename TOut>
+template <int HD, typename TOut, bool MAPS>
 int launch_mma(const void* q, int q_stride, int q_col, const int* row_slot, const int* row_pos,
                const NbPagedKV& kv, int group, void* out, int out_stride, float scale, float softcap, const float* sink, NbAttnOpts opt,
                int n_rows, int n_splits, float* part_acc, float* part_ml, int* counters, int append,
@@ -792,10 +793,10 @@ int launch_mma(const void* q, int q_stride, int q_col, const int* row_slot, cons
   long long per_sm = (long long)((228 * 1024) / (smem4 + 1024));
   if (per_sm > 8) per_sm = 8;   // 2,048 threads an SM
   if (ctas <= per_sm * sms)
-    return launch_mma_s<HD, TOut, 4, 8>(q, q_stride, q_col, row_slot, row_pos, kv, group, out, out_stride,
+    return launch_mma_s<HD, TOut, 4, 8, MAPS>(q, q_stride, q_col, row_slot, row_pos, kv, group, out, out_stride,
                                         scale, softcap, sink, opt, n_rows, n_splits, part_acc, part_ml, counters,
                                         append, k_col, v_col, clustered, stream);
-  return launch_mma_s<HD, TOut, 2, 4>(q, q_stride, q_col, row_slot, row_pos, kv, group, out, out_stride,
+  return launch_mma_s<HD, TOut, 2, 4, MAPS>(q, q_stride, q_col, row_slot, row_pos, kv, group, out, out_stride,
                                       scale, softcap, sink, opt, n_rows, n_splits, part_acc, part_ml, counters, append,
                                       k_col, v_col, clustered, stream);
 }
@@ -805,12 +806,25 @@ int mma_by_head_dim(int hd, const void* q, int q_stride, int q_col, const int* r
                     const int* row_pos, const NbPagedKV& kv, int group, void* out, int out_stride,
                     float scale, float softcap, const float* sink, NbAttnOpts opt, int n_rows, int n_splits, float* pa, float* pm,
                     int* cn, int ap, int kc, int vc, bool clustered, cudaStream_t st) {
+#define NB_ARGS q, q_stride, q_col, row_slot, row_pos, kv, group, out, out_stride, scale, softcap, sink, opt, n_rows, n_splits, pa, pm, cn, ap, kc, vc, clustered, st
+  if constexpr (sizeof(TOut) == 2) {
+    if (opt.maps) {
+      switch (hd) {
+        case 32: return launch_mma<32, TOut, true>(NB_ARGS);
+        case 64: return launch_mma<64, TOut, true>(NB_ARGS);
+        case 96: return launch_mma<96, TOut, true>(NB_ARGS);
+        case 128: return launch_mma<128, TOut, true>(NB_ARGS);
+      }
+      return NB_ERR_UNSUPPORTED;
+    }
+  }
 #define NB_HD(HD_) \
-  case HD_: return launch_mma<HD_, TOut>(q, q_stride, q_col, row_slot, row_pos, kv, group, out, out_stride, scale, softcap, sink, opt, n_rows, n_splits, pa, pm, cn, ap, kc, vc, clustered, st)
+  case HD_: return launch_mma<HD_, TOut, false>(NB_ARGS)
   switch (hd) {
     NB_HD(16); NB_HD(32); NB_HD(48); NB_HD(64); NB_HD(80); NB_HD(96); NB_HD(112); NB_HD(128);
   }
 #undef NB_HD
+#undef NB_ARGS
   return NB_ERR_UNSUPPORTED;
 }
 
