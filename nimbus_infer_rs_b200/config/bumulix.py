@@ -24,7 +24,7 @@ another.  ``attention`` is the difference of two attention maps per head over a 
 (every earlier token), ``rot.dims`` (= rot_dim), ``rot.scaling`` (none), ``streams`` (no
 connections between streams: one ordinary residual), ``residual_mult`` (1), ``logit_softcap``
 (none).  A layer with ``weights_of: j`` has no tensors of its own and runs with layer ``j``'s (its
-own cache); the rest of its entry equals layer ``j``'s.
+own cache) and must be described as that layer is.
 """
 from __future__ import annotations
 

@@ -1,8 +1,8 @@
 // Several residual streams side by side (hyper-connections), fp32, row by row:
 //
 //   u_r   = sum_s in[s] x_r[s]                              what a sublayer reads (then normed)
-//   x_r[t] <- sum_s mix[s][t] x_r[s] + gain[t] * ls * y_r    its result y written back, all streams
-//                                                           at once from the old ones
+//   x_r[t] <- sum_s mix[s][t] x_r[s] + gain[t] * ls * y_r    its result y written back (the right
+//                                                           side holds the streams as they were)
 //
 // One kernel does the write-back of a sublayer and, in the same pass over the row, what the next
 // reader of the streams wants: the RMS-normed sum u of the next sublayer (statistics in fp32 over

@@ -41,7 +41,7 @@ def read_streams(xs, coef):
 
 
 def write_streams(xs, mix, gain, y, m):
-    """All streams at once from the old ones: stream t becomes sum_s mix[s, t] xs[s] + m gain[t] y."""
+    """What the streams become, computed from what they were: stream t is sum_s mix[s, t] xs[s] + m gain[t] y."""
     S = xs.shape[0]
     new = []
     for t in range(S):
