@@ -5,7 +5,9 @@ size and window) form a *group* with a page pool, block tables and tensors of it
 
     storage[layer_in_group][0=keys | 1=values][page][kv_head][token_in_page][head_dim]
 
-(a request for one plane has no values: its mixer keeps one vector per token and head)
+(a request for one plane has no values: its mixer keeps one vector per token and head; where
+values have a size of their own the two planes of a layer lie one behind the other as
+``[page][kv_head][token_in_page][size]`` each)
 
 A page holds ``PAGE`` consecutive tokens of one sequence, for every layer of the group at
 once, so a sequence's block table (its list of pages) is shared by the group's layers.  One
@@ -50,6 +52,11 @@ class LayerKV:
     n_kv_heads: int
     head_dim: int
     window: int = 0
+    value_dim: int | None = None    # None: values have the keys' size
+
+    @property
+    def value_size(self) -> int:
+        return self.head_dim if self.value_dim is None else self.value_dim
 
 
 class PagePool:
@@ -93,9 +100,14 @@ class CacheGroup:
         if request.every < 1 or (request.every > 1 and request.window):
             raise ValueError(f"a cache request has an entry per token or per block of tokens "
                              f"without a window, not {request}")
-        self.storage = torch.zeros(
-            (len(self.layers), request.planes, n_pages, request.n_kv_heads, PAGE, request.head_dim),
-            dtype=dtype, device=device)
+        if request.planes == 1 and request.value_dim is not None:
+            raise ValueError("a store of one plane has no values of another size")
+        # values of another size than keys: a layer's two planes lie one behind the other
+        self.rows = n_pages * request.n_kv_heads * PAGE
+        self.mixed = request.planes == 2 and request.value_size != request.head_dim
+        shape = (self.rows * (request.head_dim + request.value_size),) if self.mixed else \
+            (request.planes, n_pages, request.n_kv_heads, PAGE, request.head_dim)
+        self.storage = torch.zeros((len(self.layers), *shape), dtype=dtype, device=device)
         self.block_table = torch.zeros((n_slots, self.max_pages), dtype=torch.int32, device=device)
         self._table_host = np.zeros((n_slots, self.max_pages), dtype=np.int32)
         self._pages: dict[int, list[int]] = {}   # slot -> page of every page index (-1: given back)
@@ -159,5 +171,10 @@ class CacheGroup:
     def layer_view(self, layer: int) -> LayerKV:
         i = self.layers.index(layer)
         r = self.request
+        if self.mixed:
+            shape, cut = (self.pool.n_pages, r.n_kv_heads, PAGE), self.rows * r.head_dim
+            flat = self.storage[i]
+            return LayerKV(flat[:cut].view(*shape, r.head_dim), flat[cut:].view(*shape, r.value_size),
+                           self.block_table, PAGE, r.n_kv_heads, r.head_dim, r.window, r.value_size)
         return LayerKV(self.storage[i, 0], self.storage[i, 1] if r.planes > 1 else None,
                        self.block_table, PAGE, r.n_kv_heads, r.head_dim, r.window)

@@ -11,8 +11,9 @@
 //                           plane of the paged store, and the key AS PROJECTED (no norm, no
 //                           rotation) into the V plane: the values are the keys.
 //   nb_qkv_norm_rope_append the same with values from columns of their own (any head size, a
-//                           plane and block table of their own) and the norm optional: what any
-//                           attention with rotated, optionally normed queries and keys needs.
+//                           plane and block table of their own) and the norm optional, per head
+//                           or over all heads of a row at once: what any attention with rotated,
+//                           optionally normed queries and keys needs.
 //   nb_pool_blocks          for every row that completes a block of `pool` tokens: the mean of
 //                           the block's keys as the store holds them, and of its values, into
 //                           entry pos / pool of a second paged store.
@@ -24,6 +25,7 @@
 namespace {
 
 constexpr int QK_THREADS = 128;
+constexpr int QK_PAIRS = 128;      // rotated pairs whose cos and sin a CTA keeps for all its heads
 
 template <typename TQ, typename TC>
 __global__ void __launch_bounds__(QK_THREADS)
@@ -33,9 +35,10 @@ qk_norm_rope_append_kernel(const float* src, int stride, int q_col, int k_col, i
                            const int* row_slot, const int* row_pos, TQ* q_out, TC* kc, TC* vc,
                            const int* block_table, int max_pages, const int* v_table,
                            int v_max_pages, int page, int n_heads, int n_kv_heads, int d, int dv,
-                           int write) {
+                           int write, int whole) {
   nb_grid_dependency_wait();
   nb_launch_dependents();
+  __shared__ float cos_s[QK_PAIRS], sin_s[QK_PAIRS], red[32];
   const int r = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int slot = row_slot[r];
   TQ* qo = q_out + (size_t)r * n_heads * d;
@@ -53,13 +56,36 @@ qk_norm_rope_append_kernel(const float* src, int stride, int q_col, int k_col, i
     const int v_page = v_table[(size_t)slot * v_max_pages + pos / page];
     v_row = (size_t)v_page * n_kv_heads * page + (pos % page);
   }
+  // the row's cos and sin, once for all heads
+  const bool kept = half <= QK_PAIRS;
+  if (kept)
+    for (int i = threadIdx.x; i < half; i += QK_THREADS) {
+      float s, c;
+      sincosf((float)pos * freq[i], &s, &c);
+      sin_s[i] = s * amplitude;
+      cos_s[i] = c * amplitude;
+    }
+  // norms over all heads of the row
+  float inv_q = 1.0f, inv_k = 1.0f;
+  if (whole) {
+    float sq = 0.0f, sk = 0.0f;
+    for (int i = threadIdx.x; i < n_heads * d; i += QK_THREADS) sq = fmaf(row[q_col + i], row[q_col + i], sq);
+    if (write)
+      for (int i = threadIdx.x; i < n_kv_heads * d; i += QK_THREADS)
+        sk = fmaf(row[k_col + i], row[k_col + i], sk);
+    inv_q = 1.0f / sqrtf(nb_block_sum(sq, red) / (float)(n_heads * d) + eps);
+    inv_k = 1.0f / sqrtf(nb_block_sum(sk, red) / (float)(n_kv_heads * d) + eps);
+  }
+  __syncthreads();
   for (int hh = warp; hh < n_heads + (write ? n_kv_heads : 0); hh += QK_THREADS / 32) {
     const bool is_q = hh < n_heads;
     const int g = hh - n_heads;
     const float* x = row + (is_q ? q_col + hh * d : k_col + g * d);
     const float* gamma = is_q ? q_gamma : k_gamma;
-    float inv = 1.0f;
-    if (gamma != nullptr) {
+    float inv = is_q ? inv_q : inv_k;
+    if (whole && gamma != nullptr) {
+      gamma += (is_q ? hh : g) * d;
+    } else if (gamma != nullptr) {
       float ss = 0.0f;
       for (int i = lane; i < d; i += 32) ss = fmaf(x[i], x[i], ss);
       ss = nb_warp_sum(ss);
@@ -74,9 +100,14 @@ qk_norm_rope_append_kernel(const float* src, int stride, int q_col, int k_col, i
         b = b * inv * gamma[i + half];
       }
       float s, c;
-      sincosf((float)pos * freq[i], &s, &c);
-      s *= amplitude;
-      c *= amplitude;
+      if (kept) {
+        s = sin_s[i];
+        c = cos_s[i];
+      } else {
+        sincosf((float)pos * freq[i], &s, &c);
+        s *= amplitude;
+        c *= amplitude;
+      }
       const float a2 = a * c - b * s, b2 = b * c + a * s;
       if (is_q) {
         qd[i] = nb_from_f32<TQ>(a2);
@@ -274,6 +305,8 @@ typedef __nv_bfloat16 bf16;
 // projected (dv = d, into `vc` by the keys' block table); else the values are columns v_col ..
 // of `src` (n_kv_heads heads of dv), written to the plane `vc`, whose pages `v_table` lists (the
 // keys' table again when keys and values share a store of two planes).
+// q_gamma / k_gamma: the norms' weights or null; whole: the norms run over all heads of a row (the
+// weights then have n_heads*d and n_kv_heads*d numbers).  write = 0: queries only (k_gamma null).
 NB_EXPORT int nb_qkv_norm_rope_append(const float* src, int stride, int q_col, int k_col, int v_col,
                                       const float* q_gamma, const float* k_gamma, float eps,
                                       const float* freq, int rot_dims, float amplitude,
@@ -281,11 +314,12 @@ NB_EXPORT int nb_qkv_norm_rope_append(const float* src, int stride, int q_col, i
                                       int q_dtype, void* kc, void* vc, int cache_dtype,
                                       const int* block_table, int max_pages, const int* v_table,
                                       int v_max_pages, int page, int n_heads, int n_kv_heads, int d,
-                                      int dv, int write, int n_rows, cudaStream_t stream) {
+                                      int dv, int write, int whole, int n_rows, cudaStream_t stream) {
   if (n_rows == 0) return 0;
   NB_REQUIRE(n_heads > 0 && n_kv_heads > 0 && d > 0 && dv > 0 && page > 0 && rot_dims >= 0 &&
                  rot_dims % 2 == 0 && rot_dims <= d && (rot_dims == 0 || freq != nullptr) &&
-                 (v_col >= 0 || dv == d) && (q_gamma == nullptr) == (k_gamma == nullptr),
+                 (v_col >= 0 || dv == d) && (!write || (q_gamma == nullptr) == (k_gamma == nullptr)) &&
+                 (!whole || q_gamma != nullptr),
              NB_ERR_BAD_ARG, "qkv_norm_rope_append: bad sizes heads=%d/%d d=%d/%d rot=%d", n_heads,
              n_kv_heads, d, dv, rot_dims);
   if (v_table == nullptr) { v_table = block_table; v_max_pages = max_pages; }
@@ -293,7 +327,7 @@ NB_EXPORT int nb_qkv_norm_rope_append(const float* src, int stride, int q_col, i
   NB_CUDA(nb_launch(qk_norm_rope_append_kernel<TQ, TC>, dim3(n_rows), dim3(QK_THREADS), 0, stream, \
                     src, stride, q_col, k_col, v_col, q_gamma, k_gamma, eps, freq, rot_dims,      \
                     amplitude, row_slot, row_pos, (TQ*)q_out, (TC*)kc, (TC*)vc, block_table,      \
-                    max_pages, v_table, v_max_pages, page, n_heads, n_kv_heads, d, dv, write))
+                    max_pages, v_table, v_max_pages, page, n_heads, n_kv_heads, d, dv, write, whole))
   switch (q_dtype * 2 + cache_dtype) {
     case 0: NB_QK(float, float); break;
     case 1: NB_QK(float, bf16); break;
@@ -319,7 +353,7 @@ NB_EXPORT int nb_qk_norm_rope_append(const float* src, int stride, int q_col, in
   return nb_qkv_norm_rope_append(src, stride, q_col, k_col, -1, q_gamma, k_gamma, eps, freq, rot_dims,
                                  amplitude, row_slot, row_pos, q_out, q_dtype, kc, vc, cache_dtype,
                                  block_table, max_pages, block_table, max_pages, page, n_heads,
-                                 n_kv_heads, d, d, write, n_rows, stream);
+                                 n_kv_heads, d, d, write, 0, n_rows, stream);
 }
 
 NB_EXPORT int nb_pool_blocks(const int* row_slot, const int* row_pos, const void* kc, const void* vc,

@@ -28,7 +28,7 @@
 //
 // A decode step (one token per sequence) is the same kernel with a chunk of one token: it reads
 // and writes the state once, which is all the memory traffic there is.
-#include "common.cuh"
+#include "delta_common.cuh"
 
 namespace {
 
@@ -196,35 +196,6 @@ delta_rule_kernel(const float* fused, int stride, int col_r, int col_k, int col_
   }
 }
 
-// out[r, h, :] = o[r, h, :] / sqrt(mean(o[r, h, :]^2) + eps) * norm_w[h, :] * sigmoid(gate logits).
-// A CTA per row, its warps over the heads; padding rows give zeros.
-template <typename TOut>
-__global__ void __launch_bounds__(128)
-delta_finish_kernel(const float* o_raw, const float* fused, int stride, int col_g,
-                    const float* __restrict__ norm_w, float eps, const int* row_slot, TOut* out,
-                    int n_heads, int d) {
-  nb_grid_dependency_wait();
-  nb_launch_dependents();
-  const int r = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int hd = n_heads * d;
-  const bool live = row_slot[r] >= 0;
-  for (int h = warp; h < n_heads; h += 4) {
-    TOut* dst = out + (size_t)r * hd + h * d;
-    if (!live) {
-      for (int j = lane; j < d; j += 32) dst[j] = nb_from_f32<TOut>(0.0f);
-      continue;
-    }
-    const float* o = o_raw + (size_t)r * hd + h * d;
-    const float* g = fused + (size_t)r * stride + col_g + h * d;
-    float ss = 0.0f;
-    for (int j = lane; j < d; j += 32) ss = fmaf(o[j], o[j], ss);
-    ss = nb_warp_sum(ss);
-    const float inv = 1.0f / sqrtf(ss / (float)d + eps);
-    for (int j = lane; j < d; j += 32)
-      dst[j] = nb_from_f32<TOut>(o[j] * inv * norm_w[h * d + j] * nb_sigmoid(g[j]));
-  }
-}
-
 template <int DP, int LPC>
 int launch(cudaStream_t stream, const float* fused, int stride, int col_r, int col_k, int col_v,
            int col_a, const float* decay_logits, const float* a_bias, float rate, float key_eps,
@@ -286,12 +257,6 @@ NB_EXPORT int nb_delta_rule(const float* fused, int stride, int col_r, int col_k
 #undef NB_DR
   if (rc != 0) return rc;
   NB_CHECK_LAUNCH("delta_rule");
-  if (out_dtype == NB_F32)
-    NB_CUDA(nb_launch(delta_finish_kernel<float>, dim3(n_rows), dim3(128), 0, stream, o_raw, fused,
-                      stride, col_g, norm_w, eps, row_slot, (float*)out, n_heads, d));
-  else
-    NB_CUDA(nb_launch(delta_finish_kernel<__nv_bfloat16>, dim3(n_rows), dim3(128), 0, stream, o_raw,
-                      fused, stride, col_g, norm_w, eps, row_slot, (__nv_bfloat16*)out, n_heads, d));
-  NB_CHECK_LAUNCH("delta_finish");
-  return 0;
+  return launch_delta_finish(o_raw, fused, stride, col_g, norm_w, d, eps, row_slot, out, out_dtype,
+                             n_heads, d, n_rows, stream);
 }

@@ -1,9 +1,10 @@
 // A feed-forward of routed experts: every token is run through `top` of `n_experts` small
 // gated feed-forwards and the results are added up with per-token weights.
 //
-//   nb_moe_route    scores = softmax(router logits) over all experts (fp32); the `top`
-//                   largest per row (of equal scores the lower index), with their scores as
-//                   weights (optionally renormalised to sum 1)
+//   nb_moe_route    scores = softmax(router logits, plus a bias per expert) over all experts
+//                   (fp32); the `top` largest per row (of equal scores the lower index), with
+//                   their scores as weights (optionally renormalised to sum 1, which makes them
+//                   the softmax over the chosen logits)
 //   nb_moe_route_sigmoid  scores = sigmoid(logits); chosen by score + bias among the experts of
 //                   the best groups; weights are the scores, renormalised and scaled
 //   nb_moe_group    the (row, choice) pairs grouped by expert: offsets[e] .. offsets[e+1] are
@@ -11,7 +12,8 @@
 //   nb_moe_gemm     a product per expert over its group of rows, tiled; with two weight
 //                   sets it gives act(x Wa^T) * (x Wb^T) (the gated first half of an expert),
 //                   with one the plain product (the second half)
-//   nb_moe_combine  residual[row] += sum_k weight[row, k] * y[place[row, k]], k in order
+//   nb_moe_combine  residual[row] += sum_k weight[row, k] * y[place[row, k]], k in order; and,
+//                   where asked for, the new residual rows rounded to another type
 //
 // Everything is read from device memory (no count comes back to the host), so a step with
 // routed experts can be recorded in a CUDA graph.  A row's result does not depend on where
@@ -48,7 +50,9 @@ __device__ __forceinline__ void route_take_best(float (&v)[PL], int lane, float 
     if (lane + 32 * i == best_e) v[i] = neg;
 }
 
-__global__ void moe_route_kernel(const float* logits, int stride, int col, const int* row_slot,
+template <int PL>   // experts a lane holds: n_experts <= 32 * PL
+__global__ void moe_route_kernel(const float* logits, int stride, int col,
+                                 const float* __restrict__ bias, const int* row_slot,
                                  int n_rows, int n_experts, int top, int renormalize, int* idx,
                                  float* weight) {
   nb_grid_dependency_wait();
@@ -64,18 +68,18 @@ __global__ void moe_route_kernel(const float* logits, int stride, int col, const
     return;
   }
   const float* z = logits + (size_t)r * stride + col;
-  float v[ROUTE_MAX_PER_LANE];
+  float v[PL];
   float m = -INFINITY;
 #pragma unroll
-  for (int i = 0; i < ROUTE_MAX_PER_LANE; ++i) {
+  for (int i = 0; i < PL; ++i) {
     const int e = lane + 32 * i;
-    v[i] = e < n_experts ? z[e] : -INFINITY;
+    v[i] = e < n_experts ? z[e] + (bias != nullptr ? bias[e] : 0.0f) : -INFINITY;
     m = fmaxf(m, v[i]);
   }
   m = nb_warp_max(m);
   float sum = 0.0f;
 #pragma unroll
-  for (int i = 0; i < ROUTE_MAX_PER_LANE; ++i) {
+  for (int i = 0; i < PL; ++i) {
     const int e = lane + 32 * i;
     v[i] = e < n_experts ? expf(v[i] - m) : -1.0f;   // scores are >= 0; -1 marks "none"/"taken"
     if (e < n_experts) sum += v[i];
@@ -321,8 +325,9 @@ moe_gemm_kernel(const TX* x, int x_stride, const int* order, int row_div, const 
   }
 }
 
+template <typename TO>
 __global__ void moe_combine_kernel(const float* y, int width, const int* place, const float* weight,
-                                   int top, float* residual) {
+                                   int top, float* residual, TO* out_cast) {
   nb_grid_dependency_wait();
   nb_launch_dependents();
   const int r = blockIdx.x;
@@ -332,7 +337,9 @@ __global__ void moe_combine_kernel(const float* y, int width, const int* place, 
       const int at = place[(size_t)r * top + k];
       if (at >= 0) s = fmaf(weight[(size_t)r * top + k], y[(size_t)at * width + i], s);
     }
-    residual[(size_t)r * width + i] += s;
+    s += residual[(size_t)r * width + i];
+    residual[(size_t)r * width + i] = s;
+    if (out_cast != nullptr) out_cast[(size_t)r * width + i] = nb_from_f32<TO>(s);
   }
 }
 
@@ -340,17 +347,24 @@ __global__ void moe_combine_kernel(const float* y, int width, const int* place, 
 
 typedef __nv_bfloat16 bf16;
 
-NB_EXPORT int nb_moe_route(const float* logits, int stride, int col, const int* row_slot, int n_rows,
-                           int n_experts, int top, int renormalize, int* idx, float* weight,
-                           cudaStream_t stream) {
+// bias: fp32 [n_experts] or null.
+NB_EXPORT int nb_moe_route(const float* logits, int stride, int col, const float* bias,
+                           const int* row_slot, int n_rows, int n_experts, int top, int renormalize,
+                           int* idx, float* weight, cudaStream_t stream) {
   if (n_rows == 0) return 0;
   NB_REQUIRE(n_experts >= 1 && n_experts <= 32 * ROUTE_MAX_PER_LANE, NB_ERR_UNSUPPORTED,
              "moe_route: %d experts are outside 1..%d", n_experts, 32 * ROUTE_MAX_PER_LANE);
   NB_REQUIRE(top >= 1 && top <= n_experts, NB_ERR_BAD_ARG, "moe_route: top=%d of %d experts", top,
              n_experts);
   NB_REQUIRE(col >= 0 && stride >= col + n_experts, NB_ERR_BAD_ARG, "moe_route: bad columns");
-  NB_CUDA(nb_launch(moe_route_kernel, dim3((n_rows + 3) / 4), dim3(128), 0, stream, logits, stride,
-                    col, row_slot, n_rows, n_experts, top, renormalize, idx, weight));
+#define NB_RT(PL_)                                                                               \
+  NB_CUDA(nb_launch(moe_route_kernel<PL_>, dim3((n_rows + 3) / 4), dim3(128), 0, stream, logits, \
+                    stride, col, bias, row_slot, n_rows, n_experts, top, renormalize, idx, weight))
+  if (n_experts <= 32) NB_RT(1);
+  else if (n_experts <= 64) NB_RT(2);
+  else if (n_experts <= 256) NB_RT(8);
+  else NB_RT(ROUTE_MAX_PER_LANE);
+#undef NB_RT
   NB_CHECK_LAUNCH("moe_route");
   return 0;
 }
@@ -440,16 +454,22 @@ NB_EXPORT int nb_moe_gemm(const void* x, int x_dtype, int x_stride, const int* o
   return 0;
 }
 
+// out_cast (or null): [n_rows][width] of cast_dtype, the residual rows as they then are.
 NB_EXPORT int nb_moe_combine(const float* y, int width, const int* place, const float* weight,
-                             int top, float* residual, int n_rows, cudaStream_t stream) {
+                             int top, float* residual, void* out_cast, int cast_dtype, int n_rows,
+                             cudaStream_t stream) {
   if (n_rows == 0) return 0;
   NB_REQUIRE(width > 0 && top >= 1, NB_ERR_BAD_ARG, "moe_combine: bad sizes");
   // a thread per element of the stream while the launch stays small; rows of a long prompt
   // walk over their width instead
   const int threads = 128;
   const int chunks = n_rows <= 256 ? (width + threads - 1) / threads : (width + 4 * threads - 1) / (4 * threads);
-  NB_CUDA(nb_launch(moe_combine_kernel, dim3(n_rows, chunks), dim3(threads), 0, stream, y, width,
-                    place, weight, top, residual));
+  if (out_cast != nullptr && cast_dtype == NB_BF16)
+    NB_CUDA(nb_launch(moe_combine_kernel<bf16>, dim3(n_rows, chunks), dim3(threads), 0, stream, y,
+                      width, place, weight, top, residual, (bf16*)out_cast));
+  else
+    NB_CUDA(nb_launch(moe_combine_kernel<float>, dim3(n_rows, chunks), dim3(threads), 0, stream, y,
+                      width, place, weight, top, residual, (float*)out_cast));
   NB_CHECK_LAUNCH("moe_combine");
   return 0;
 }

@@ -198,6 +198,7 @@ moe_mma_kernel(const TX* x, int x_stride, const int* order, int row_div, const i
   const int g = lane >> 2, t4 = lane & 3;
   // neighbouring 16-bit results leave together when every row starts on a 4-byte boundary
   const bool pairs = sizeof(TY) == 2 && y_stride % 2 == 0 && (reinterpret_cast<uintptr_t>(y) & 3) == 0;
+  const bool pairs4 = sizeof(TY) == 4 && y_stride % 2 == 0 && (reinterpret_cast<uintptr_t>(y) & 7) == 0;
 #pragma unroll
   for (int mi = 0; mi < MI; ++mi) {
 #pragma unroll
@@ -231,6 +232,8 @@ moe_mma_kernel(const TX* x, int x_stride, const int* order, int row_div, const i
         TY* dst = y + (size_t)p * y_stride + n;
         if (sizeof(TY) == 2 && pairs && n + 1 < N) {
           *reinterpret_cast<uint32_t*>(dst) = pack_bf16(v[0], v[1]);
+        } else if (sizeof(TY) == 4 && pairs4 && n + 1 < N) {
+          *reinterpret_cast<float2*>(dst) = make_float2(v[0], v[1]);
         } else {
           if (n < N) dst[0] = nb_from_f32<TY>(v[0]);
           if (n + 1 < N) dst[1] = nb_from_f32<TY>(v[1]);
@@ -312,20 +315,20 @@ NB_EXPORT int nb_moe_gemm_mma(const void* x, int x_stride, const int* order, int
   return 0;
 }
 
-// The per-head linear map (the contract of nb_head_linear) for bf16 weights and bf16 results;
-// x: bf16 or fp32 rows (fp32 is rounded to bf16 on the way in).
+// The per-head linear map (the contract of nb_head_linear) for bf16 weights and bf16 or
+// fp32 results; x: bf16 or fp32 rows (fp32 is rounded to bf16 on the way in).
 NB_EXPORT int nb_head_linear_mma_supported(int x_dtype, int w_dtype, int y_dtype, int x_stride,
                                            int x_col, int n_in) {
-  return w_dtype == NB_BF16 && y_dtype == NB_BF16 && n_in % 8 == 0 &&
+  return w_dtype == NB_BF16 && (y_dtype == NB_BF16 || y_dtype == NB_F32) && n_in % 8 == 0 &&
          (x_dtype == NB_F32 || (x_dtype == NB_BF16 && x_stride % 8 == 0 && x_col % 8 == 0));
 }
 
 NB_EXPORT int nb_head_linear_mma(const void* x, int x_dtype, int x_stride, int x_col, const void* W,
-                                 void* y, int y_stride, int y_hstride, const float* gate,
+                                 void* y, int y_dtype, int y_stride, int y_hstride, const float* gate,
                                  int gate_stride, int gate_col, int gate_each, const int* row_slot,
                                  int n_rows, int n_heads, int n_in, int n_out, cudaStream_t stream) {
   if (n_rows == 0) return 0;
-  NB_REQUIRE(nb_head_linear_mma_supported(x_dtype, NB_BF16, NB_BF16, x_stride, x_col, n_in),
+  NB_REQUIRE(nb_head_linear_mma_supported(x_dtype, NB_BF16, y_dtype, x_stride, x_col, n_in),
              NB_ERR_UNSUPPORTED, "head_linear_mma: shape not supported (in=%d stride=%d col=%d)", n_in,
              x_stride, x_col);
   NB_REQUIRE((uintptr_t)W % 16 == 0 && (x_dtype == NB_F32 || (uintptr_t)x % 16 == 0), NB_ERR_BAD_ARG,
@@ -334,15 +337,21 @@ NB_EXPORT int nb_head_linear_mma(const void* x, int x_dtype, int x_stride, int x
   u.rows = n_rows; u.x_gcol = n_in; u.y_gcol = y_hstride; u.row_slot = row_slot;
   u.gate = gate; u.gate_stride = gate_stride; u.gate_col = gate_col; u.gate_each = gate_each;
   int rc;
-#define NB_GO(S_, TX_)                                                                               \
-  rc = launch<S_, false, TX_, bf16>(((n_rows + S_::BM - 1) / S_::BM) * n_heads, stream,               \
+#define NB_GO(S_, TX_, TY_)                                                                          \
+  rc = launch<S_, false, TX_, TY_>(((n_rows + S_::BM - 1) / S_::BM) * n_heads, stream,               \
                                     (const TX_*)x + x_col, x_stride, nullptr, 1, nullptr, n_heads,    \
-                                    (const bf16*)W, nullptr, (bf16*)y, y_stride, n_out, n_in, 0, 0.0f, u)
+                                    (const bf16*)W, nullptr, (TY_*)y, y_stride, n_out, n_in, 0, 0.0f, u)
+#define NB_GO_Y(S_, TX_)                                                                             \
+  do {                                                                                               \
+    if (y_dtype == NB_F32) NB_GO(S_, TX_, float);                                                    \
+    else NB_GO(S_, TX_, bf16);                                                                       \
+  } while (0)
   if (n_rows <= 16) {
-    if (x_dtype == NB_F32) NB_GO(Small, float); else NB_GO(Small, bf16);
+    if (x_dtype == NB_F32) NB_GO_Y(Small, float); else NB_GO_Y(Small, bf16);
   } else {
-    if (x_dtype == NB_F32) NB_GO(Large, float); else NB_GO(Large, bf16);
+    if (x_dtype == NB_F32) NB_GO_Y(Large, float); else NB_GO_Y(Large, bf16);
   }
+#undef NB_GO_Y
 #undef NB_GO
   if (rc) return rc;
   NB_CHECK_LAUNCH("head_linear_mma");

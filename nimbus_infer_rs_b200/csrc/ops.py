@@ -674,7 +674,7 @@ class CudaBackend:
         if self.use_mma and self.lib.nb_head_linear_mma_supported(
                 dtype_code(x.dtype), dtype_code(w.dtype), dtype_code(out.dtype), x.shape[1], x_col, n_in):
             self._call("nb_head_linear_mma", _ptr(x), dtype_code(x.dtype), x.shape[1], x_col, _ptr(w),
-                       _ptr(out), out.shape[1], pitch, _ptr(gate),
+                       _ptr(out), dtype_code(out.dtype), out.shape[1], pitch, _ptr(gate),
                        gate.shape[1] if gate is not None else 0, gate_col, 1 if gate_each else 0,
                        _ptr(layout.row_slot), n, n_heads, n_in, n_out, self._stream())
             return
@@ -782,11 +782,17 @@ class CudaBackend:
                    kv.block_table.shape[1], kv.page, n_heads, G, d, 1 if write else 0, n,
                    self._stream())
 
+    @staticmethod
+    def _value_size(k_store, v_store):
+        """Numbers of a value: of the V plane when one store holds both, else of the store of values."""
+        return k_store.value_size if v_store is k_store else v_store.head_dim
+
     def qkv_norm_rope_append(self, src, q_col, k_col, v_col, q_gamma, k_gamma, eps, freq, rot_dims,
-                             amplitude, layout, k_store, v_store, n_heads, value_dim, q_out, write):
-        """Queries, keys and values of the fp32 rows ``src`` made ready: per head an optional RMS
-        norm (``q_gamma`` / ``k_gamma`` or ``None``) and the rotation of the first ``rot_dims``
-        numbers of queries and keys; queries to ``q_out``, keys to the K plane of ``k_store``,
+                             amplitude, layout, k_store, v_store, n_heads, value_dim, q_out, write,
+                             whole=False):
+        """Queries, keys and values of the fp32 rows ``src`` made ready: an optional RMS norm
+        (``q_gamma`` / ``k_gamma`` or ``None``) per head, or with ``whole`` over all heads at once,
+        and the rotation of the first ``rot_dims`` numbers of queries and keys; queries to ``q_out``, keys to the K plane of ``k_store``,
         values (columns ``v_col ..``, heads of ``value_dim``) to the V plane of ``k_store`` when
         ``v_store`` is the same store, else to the one plane of ``v_store``."""
         _check(src, "src", torch.float32, 2)
@@ -795,10 +801,14 @@ class CudaBackend:
         n = layout.n_rows
         shared = v_store is k_store
         v_plane = k_store.v if shared else v_store.k
+        q_norm, k_norm = (n_heads * d, G * d) if whole else (d, d)
         if q_out.shape != (n, n_heads * d) or src.shape[0] < n or v_plane is None or \
-                src.shape[1] < max(q_col + n_heads * d, k_col + G * d, v_col + G * value_dim) or \
-                v_store.head_dim != value_dim or v_store.n_kv_heads != G or \
-                (q_gamma is not None and (q_gamma.numel() != d or k_gamma.numel() != d)) or \
+                src.shape[1] < max(q_col + n_heads * d,
+                                   max(k_col + G * d, v_col + G * value_dim) if write else 0) or \
+                self._value_size(k_store, v_store) != value_dim or v_store.n_kv_heads != G or \
+                (q_gamma is not None and q_gamma.numel() != q_norm) or \
+                (write and (q_gamma is None) != (k_gamma is None)) or \
+                (k_gamma is not None and k_gamma.numel() != k_norm) or \
                 (rot_dims and (freq is None or freq.numel() != rot_dims // 2)):
             raise KernelError("qkv_norm_rope_append: shapes do not agree")
         self._call("nb_qkv_norm_rope_append", _ptr(src), src.shape[1], q_col, k_col, v_col,
@@ -808,7 +818,7 @@ class CudaBackend:
                    dtype_code(k_store.k.dtype), _ptr(k_store.block_table),
                    k_store.block_table.shape[1], _ptr(v_store.block_table),
                    v_store.block_table.shape[1], k_store.page, n_heads, G, d, value_dim,
-                   1 if write else 0, n, self._stream())
+                   1 if write else 0, 1 if whole else 0, n, self._stream())
 
     def attention_masked(self, q, layout, k_store, v_store, n_heads, sink, out, scale, softcap=0.0,
                          window=0, keep_first=0, chunk=0, gate=None, gate_col=0):
@@ -819,7 +829,7 @@ class CudaBackend:
         head ``h``'s result is multiplied by ``sigmoid`` of it."""
         _check(q, "q", None, 2)
         _check(out, "out", None, 2)
-        n, d, dv = layout.n_rows, k_store.head_dim, v_store.head_dim
+        n, d, dv = layout.n_rows, k_store.head_dim, self._value_size(k_store, v_store)
         shared = v_store is k_store
         if q.shape != (n, n_heads * d) or out.shape != (n, n_heads * dv) or \
                 k_store.n_kv_heads != v_store.n_kv_heads or k_store.k.dtype != v_store.k.dtype or \
@@ -836,7 +846,8 @@ class CudaBackend:
         look_back = window if window > 0 else chunk
         keeps = window > 0 and keep_first > 0
         code = dtype_code(q.dtype)
-        if shared and q.dtype == k_store.k.dtype and layout.is_decode and \
+        one_size = shared and d == dv
+        if one_size and q.dtype == k_store.k.dtype and layout.is_decode and \
                 self.lib.nb_attention_decode_supported(code, d, n_heads, k_store.n_kv_heads, k_store.page) \
                 and (q.dtype != torch.bfloat16 or q.shape[1] % 8 == 0):
             # one-token steps: the split decode kernel; kept first tokens are its last split, the
@@ -854,7 +865,7 @@ class CudaBackend:
                        int(chunk), _ptr(gate), gate.shape[1] if gate is not None else 0, int(gate_col),
                        n, n_splits, _ptr(acc), _ptr(ml), _ptr(counters), self._stream())
             return
-        if shared and q.dtype == k_store.k.dtype and not layout.is_decode and self.use_tcgen05 \
+        if one_size and q.dtype == k_store.k.dtype and not layout.is_decode and self.use_tcgen05 \
                 and scale > 0 and self.lib.nb_attention_prefill_tc_supported(
                     code, d, n_heads, k_store.n_kv_heads, k_store.page, q.shape[1], 0,
                     dtype_code(out.dtype), out.shape[1]):
@@ -886,7 +897,7 @@ class CudaBackend:
                        layout.n_seqs, layout.max_q_len, max_splits, per_run, _ptr(part),
                        _ptr(counters), 0, 0, 0, self._stream())
             return
-        if shared and q.dtype == torch.bfloat16 and k_store.k.dtype == torch.bfloat16 \
+        if one_size and q.dtype == torch.bfloat16 and k_store.k.dtype == torch.bfloat16 \
                 and not layout.is_decode and self.use_mma and self.lib.nb_attention_prefill_supported(
                     code, d, n_heads, k_store.n_kv_heads, k_store.page, q.shape[1], 0):
             # prompts in bfloat16 with other heads (16, 32, 48, 96; 64 and 128 when tcgen05 is
@@ -1045,6 +1056,40 @@ class CudaBackend:
                    _ptr(state), _ptr(o_raw), _ptr(out), dtype_code(out.dtype), n_heads, dim,
                    layout.n_seqs, n, self._stream())
         self.launches += 1
+
+    def gated_delta(self, qkv, beta, col_beta, low, col_decay, col_gate, a_log, dt_bias, norm, eps,
+                    key_eps, layout, state, n_heads, n_kv_heads, d, dv, out):
+        """The gated delta rule over each sequence's rows in order, from and into the sequences'
+        state rows (``state``: fp32 ``[slots, n_heads * d * dv]``).  ``qkv``: convolved and activated
+        rows ``[q | k | v]`` (``n_kv_heads``, ``n_kv_heads`` and ``n_heads`` heads); ``beta``: rows with
+        the heads' logits at ``col_beta``; ``low``: rows with the decay logits at ``col_decay`` and the
+        output gate's at ``col_gate``; all fp32.  The heads' outputs normed, weighted and gated
+        into ``out``."""
+        for t, nm in ((qkv, "qkv"), (beta, "beta"), (low, "low")):
+            _check(t, nm, torch.float32, 2)
+        _check(out, "out", None, 2)
+        n, H, G = layout.n_rows, n_heads, n_kv_heads
+        if out.shape != (n, H * dv) or qkv.shape[0] < n or qkv.shape[1] != 2 * G * d + H * dv or \
+                beta.shape[0] < n or beta.shape[1] < col_beta + H or low.shape[0] < n or \
+                low.shape[1] < max(col_decay + H * d, col_gate + H * dv) or a_log.numel() != H or \
+                dt_bias.numel() != H * d or norm.numel() != dv:
+            raise KernelError("gated_delta: shapes do not agree")
+        st = self._state_rows(state, H * d * dv)
+        args = (_ptr(qkv), qkv.shape[1], _ptr(beta), beta.shape[1], col_beta, _ptr(low), low.shape[1],
+                col_decay, col_gate, _ptr(a_log), _ptr(dt_bias), _ptr(norm), float(eps), float(key_eps),
+                _ptr(layout.cu_rows), _ptr(layout.seq_slot))
+        if layout.is_decode and layout.max_q_len == 1:
+            self._call("nb_gated_delta_step", *args, _ptr(st), st.stride(0), _ptr(out),
+                       dtype_code(out.dtype), H, G, d, dv, layout.n_seqs, self._stream())
+            return
+        # what every block of four tokens does to the state, and the outputs before their norm
+        records = torch.empty(self.lib.nb_gated_delta_scratch(n, layout.n_seqs, H, d, dv),
+                              device=out.device, dtype=torch.float32)
+        o_raw = torch.empty((n, H * dv), device=out.device, dtype=torch.float32)
+        self._call("nb_gated_delta", *args, _ptr(layout.row_slot), _ptr(st), st.stride(0),
+                   _ptr(records), _ptr(o_raw), _ptr(out), dtype_code(out.dtype), H, G, d, dv,
+                   layout.n_seqs, layout.max_q_len, n, self._stream())
+        self.launches += 2
 
     # -- short convolutions, capped attention, linear recurrences ------------------------
     @staticmethod
@@ -1215,16 +1260,33 @@ class CudaBackend:
                    float(next_eps), _ptr(out_next),
                    dtype_code(out_next.dtype) if out_next is not None else 0, n, d, self._stream())
 
-    def glu_rows(self, x, gate_col, up_col, act, out, act_param=0.0):
+    def scaled_pair_add(self, a, scale_a, b, scale_b, residual, next_gamma=None, next_eps=0.0,
+                        out_next=None):
+        """``residual += scale_a * a + scale_b * b`` per fp32 row, and in the same pass, where asked
+        for, ``out_next = rms-norm(residual) * next_gamma``."""
+        for t, nm in ((a, "a"), (b, "b"), (residual, "residual")):
+            _check(t, nm, torch.float32, 2)
+        n, d = residual.shape
+        if a.shape != (n, d) or b.shape != (n, d) or \
+                (out_next is not None and (out_next.shape != (n, d) or next_gamma is None
+                                           or next_gamma.numel() != d)):
+            raise KernelError("scaled_pair_add: shapes do not agree")
+        self._call("nb_scaled_pair_add", _ptr(a), float(scale_a), _ptr(b), float(scale_b),
+                   _ptr(residual), _ptr(next_gamma if out_next is not None else None),
+                   float(next_eps), _ptr(out_next),
+                   dtype_code(out_next.dtype) if out_next is not None else 0, n, d, self._stream())
+
+    def glu_rows(self, x, gate_col, up_col, act, out, act_param=0.0, row_gate_col=-1):
         """``out[r, i] = act(x[r, gate_col + i]) * x[r, up_col + i]`` for fp32 rows ``x`` (or the
-        combiner of ``ACT_SWISH_CLAMP`` with its bound ``act_param``)."""
+        combiner of ``ACT_SWISH_CLAMP`` with its bound ``act_param``); ``row_gate_col`` >= 0: times
+        ``sigmoid(x[r, row_gate_col])``."""
         _check(x, "x", torch.float32, 2)
         _check(out, "out", None, 2)
         n, d = out.shape
-        if x.shape[0] < n or x.shape[1] < max(gate_col, up_col) + d:
+        if x.shape[0] < n or x.shape[1] < max(gate_col, up_col) + d or x.shape[1] <= row_gate_col:
             raise KernelError("glu_rows: shapes do not agree")
         self._call("nb_glu_rows", _ptr(x), x.shape[1], gate_col, up_col, int(act), float(act_param),
-                   _ptr(out), dtype_code(out.dtype), n, d, self._stream())
+                   int(row_gate_col), _ptr(out), dtype_code(out.dtype), n, d, self._stream())
 
     def cast_cols(self, x, out, out_col):
         """``out[:, out_col : out_col + d] = x`` (fp32 rows into columns of rows of another type)."""
@@ -1237,16 +1299,21 @@ class CudaBackend:
                    n, d, self._stream())
 
     # -- routed experts ---------------------------------------------------------------
-    def moe_route(self, logits, col, n_experts, top, renormalize, layout, idx, weight):
-        """Per row: softmax over the ``n_experts`` fp32 logits at columns ``col ..``, the ``top``
-        largest (of equal scores the lower index) into ``idx`` / ``weight`` ``[rows, top]``."""
+    def moe_route(self, logits, col, n_experts, top, renormalize, layout, idx, weight, bias=None):
+        """Per row: softmax over the ``n_experts`` fp32 logits at columns ``col ..`` (plus ``bias``,
+        a number per expert), the ``top`` largest (of equal scores the lower index) into ``idx`` /
+        ``weight`` ``[rows, top]``."""
         _check(logits, "logits", torch.float32, 2)
         _check(idx, "idx", torch.int32, 2)
         _check(weight, "weight", torch.float32, 2)
         n = layout.n_rows
         if logits.shape[0] < n or idx.shape != (n, top) or weight.shape != (n, top):
             raise KernelError("moe_route: shapes do not agree")
-        self._call("nb_moe_route", _ptr(logits), logits.shape[1], col, _ptr(layout.row_slot), n,
+        if bias is not None:
+            _check(bias, "bias", torch.float32, 1)
+            if bias.numel() != n_experts:
+                raise KernelError("moe_route: one bias per expert")
+        self._call("nb_moe_route", _ptr(logits), logits.shape[1], col, _ptr(bias), _ptr(layout.row_slot), n,
                    n_experts, top, 1 if renormalize else 0, _ptr(idx), _ptr(weight), self._stream())
 
     def moe_route_sigmoid(self, logits, col, bias, n_experts, top, n_groups, keep_groups, group_top,
@@ -1325,8 +1392,9 @@ class CudaBackend:
                    _ptr(out), dtype_code(out.dtype), out.shape[1], N, K, act, float(act_param),
                    self._stream())
 
-    def moe_combine(self, y, place, weight, residual):
-        """``residual[r] += sum_k weight[r, k] * y[place[r, k]]`` (fp32, ``k`` in order)."""
+    def moe_combine(self, y, place, weight, residual, out_cast=None):
+        """``residual[r] += sum_k weight[r, k] * y[place[r, k]]`` (fp32, ``k`` in order); ``out_cast``:
+        rows that take ``residual`` as it then is, in their own type."""
         _check(y, "y", torch.float32, 2)
         _check(place, "place", torch.int32)
         _check(weight, "weight", torch.float32, 2)
@@ -1334,8 +1402,13 @@ class CudaBackend:
         n, top = weight.shape
         if residual.shape[0] < n or residual.shape[1] != y.shape[1] or place.numel() < n * top:
             raise KernelError("moe_combine: shapes do not agree")
+        if out_cast is not None:
+            _check(out_cast, "out_cast", None, 2)
+            if out_cast.shape[0] < n or out_cast.shape[1] != y.shape[1]:
+                raise KernelError("moe_combine: out_cast shape does not match")
         self._call("nb_moe_combine", _ptr(y), y.shape[1], _ptr(place), _ptr(weight), top,
-                   _ptr(residual), n, self._stream())
+                   _ptr(residual), _ptr(out_cast),
+                   dtype_code(out_cast.dtype) if out_cast is not None else 0, n, self._stream())
 
     def advance_decode(self, tokens, next_tokens, row_pos, row_slot):
         """tokens <- next_tokens, row_pos += 1 for live rows (between two decode steps)."""

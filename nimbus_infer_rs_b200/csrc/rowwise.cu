@@ -754,11 +754,12 @@ NB_EXPORT int nb_gather_mul(const float* g, const void* table, int table_dtype, 
 
 // ---------------------------------------------------------------------------------
 // out[r, i] = act(x[r, gate_col + i]) * x[r, up_col + i] (nb_gate_up): the gated half of a feed-forward whose
-// two first products come side by side in one fp32 row.
+// two first products come side by side in one fp32 row.  row_gate_col >= 0: times
+// sigmoid(x[r, row_gate_col]), one number per row.
 // ---------------------------------------------------------------------------------
 template <typename TOut>
 __global__ void glu_rows_kernel(const float* x, int x_stride, int gate_col, int up_col, int act,
-                                float act_param, TOut* out, int d, size_t total) {
+                                float act_param, int row_gate_col, TOut* out, int d, size_t total) {
   nb_grid_dependency_wait();
   nb_launch_dependents();
   for (size_t e = (size_t)blockIdx.x * blockDim.x + threadIdx.x; e < total;
@@ -766,26 +767,29 @@ __global__ void glu_rows_kernel(const float* x, int x_stride, int gate_col, int 
     const size_t r = e / d;
     const int i = (int)(e - r * d);
     const float* row = x + r * x_stride;
-    out[e] = nb_from_f32<TOut>(nb_gate_up<false>(row[gate_col + i], row[up_col + i], act, act_param));
+    float v = nb_gate_up<false>(row[gate_col + i], row[up_col + i], act, act_param);
+    if (row_gate_col >= 0) v *= nb_sigmoid(row[row_gate_col]);
+    out[e] = nb_from_f32<TOut>(v);
   }
 }
 
 NB_EXPORT int nb_glu_rows(const float* x, int x_stride, int gate_col, int up_col, int act,
-                          float act_param, void* out, int out_dtype, int n_rows, int d,
-                          cudaStream_t stream) {
+                          float act_param, int row_gate_col, void* out, int out_dtype, int n_rows,
+                          int d, cudaStream_t stream) {
   if (n_rows == 0 || d == 0) return 0;
   NB_REQUIRE(n_rows > 0 && d > 0 && gate_col >= 0 && up_col >= 0 && x_stride >= gate_col + d &&
-                 x_stride >= up_col + d,
+                 x_stride >= up_col + d && x_stride > row_gate_col,
              NB_ERR_BAD_ARG, "glu_rows: bad sizes rows=%d d=%d cols=%d/%d stride=%d", n_rows, d,
              gate_col, up_col, x_stride);
   const size_t total = (size_t)n_rows * d;
   const int blocks = (int)((total + 1023) / 1024 < 148 * 8 ? (total + 1023) / 1024 : 148 * 8);
   if (out_dtype == NB_F32)
     NB_CUDA(nb_launch(glu_rows_kernel<float>, dim3(blocks), dim3(256), 0, stream, x, x_stride,
-                      gate_col, up_col, act, act_param, (float*)out, d, total));
+                      gate_col, up_col, act, act_param, row_gate_col, (float*)out, d, total));
   else if (out_dtype == NB_BF16)
     NB_CUDA(nb_launch(glu_rows_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, x,
-                      x_stride, gate_col, up_col, act, act_param, (__nv_bfloat16*)out, d, total));
+                      x_stride, gate_col, up_col, act, act_param, row_gate_col, (__nv_bfloat16*)out, d,
+                      total));
   else
     NB_REQUIRE(false, NB_ERR_BAD_ARG, "glu_rows: unknown output dtype %d", out_dtype);
   NB_CHECK_LAUNCH("glu_rows");
@@ -930,6 +934,110 @@ NB_EXPORT int nb_rms_pair_add(const float* a, const float* gamma_a, const float*
   else
     NB_REQUIRE(false, NB_ERR_BAD_ARG, "rms_pair_add: unknown output dtype %d", out_dtype);
   NB_CHECK_LAUNCH("rms_pair_add");
+  return 0;
+}
+
+// ---------------------------------------------------------------------------------
+// Two sublayers' results, each times a constant, into the stream, and (optionally) the norm in
+// front of the stream's next reader in the same pass:
+//   x[r] += coef_a * a[r] + coef_b * b[r]                                          (fp32)
+//   out_next[r] = x[r] / sqrt(mean(x[r]^2) + next_eps) * next_gamma    if out_next  (TOut)
+// A CTA per row, the row in registers between the two; VEC: 16 bytes a load (NV of them a thread).
+// ---------------------------------------------------------------------------------
+template <typename TOut, int NV>
+__global__ void __launch_bounds__(512)
+scaled_pair_add_vec_kernel(const float* a, float coef_a, const float* b, float coef_b, float* x,
+                           const float* __restrict__ next_gamma, float next_eps, TOut* out_next,
+                           int d) {
+  nb_grid_dependency_wait();
+  nb_launch_dependents();
+  __shared__ float red[32];
+  const size_t base = (size_t)blockIdx.x * d;
+  float4 v[NV];
+  float ss = 0.0f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int k = (threadIdx.x + i * blockDim.x) * 4;
+    v[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    if (k < d) {
+      const float4 p = *reinterpret_cast<const float4*>(a + base + k);
+      const float4 q = *reinterpret_cast<const float4*>(b + base + k);
+      v[i] = *reinterpret_cast<const float4*>(x + base + k);
+      v[i].x += fmaf(coef_a, p.x, coef_b * q.x);
+      v[i].y += fmaf(coef_a, p.y, coef_b * q.y);
+      v[i].z += fmaf(coef_a, p.z, coef_b * q.z);
+      v[i].w += fmaf(coef_a, p.w, coef_b * q.w);
+      *reinterpret_cast<float4*>(x + base + k) = v[i];
+    }
+    ss += (v[i].x * v[i].x + v[i].y * v[i].y) + (v[i].z * v[i].z + v[i].w * v[i].w);
+  }
+  if (out_next == nullptr) return;
+  ss = nb_block_sum(ss, red);
+  const float inv = 1.0f / sqrtf(ss / (float)d + next_eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int k = (threadIdx.x + i * blockDim.x) * 4;
+    if (k >= d) continue;
+    const float4 g = *reinterpret_cast<const float4*>(next_gamma + k);
+    nb_store4(out_next + base + k, v[i].x * inv * g.x, v[i].y * inv * g.y, v[i].z * inv * g.z,
+              v[i].w * inv * g.w);
+  }
+}
+
+template <typename TOut>
+__global__ void scaled_pair_add_kernel(const float* a, float coef_a, const float* b, float coef_b,
+                                       float* x, const float* __restrict__ next_gamma,
+                                       float next_eps, TOut* out_next, int d) {
+  nb_grid_dependency_wait();
+  nb_launch_dependents();
+  __shared__ float red[32];
+  const size_t base = (size_t)blockIdx.x * d;
+  float ss = 0.0f;
+  for (int i = threadIdx.x; i < d; i += blockDim.x) {
+    const float v = x[base + i] + fmaf(coef_a, a[base + i], coef_b * b[base + i]);
+    x[base + i] = v;
+    ss = fmaf(v, v, ss);
+  }
+  if (out_next == nullptr) return;
+  ss = nb_block_sum(ss, red);
+  const float inv = 1.0f / sqrtf(ss / (float)d + next_eps);
+  for (int i = threadIdx.x; i < d; i += blockDim.x)
+    out_next[base + i] = nb_from_f32<TOut>(x[base + i] * inv * next_gamma[i]);
+}
+
+template <typename TOut>
+static int launch_scaled_pair_add(const float* a, float coef_a, const float* b, float coef_b, float* x,
+                                  const float* next_gamma, float next_eps, void* out_next,
+                                  int n_rows, int d, cudaStream_t stream) {
+  const bool vec = d % 4 == 0 && d <= 4 * 512 * 4 &&
+                   ((uintptr_t)a | (uintptr_t)b | (uintptr_t)x | (uintptr_t)next_gamma |
+                    (uintptr_t)out_next) % 16 == 0;
+  const int quads = d / 4;
+#define NB_SPA(KERN, THREADS)                                                                    \
+  NB_CUDA(nb_launch(KERN, dim3(n_rows), dim3(THREADS), 0, stream, a, coef_a, b, coef_b, x,       \
+                    next_gamma, next_eps, (TOut*)out_next, d))
+  if (vec && quads <= 512) NB_SPA((scaled_pair_add_vec_kernel<TOut, 1>), (quads + 31) / 32 * 32);
+  else if (vec && quads <= 1024) NB_SPA((scaled_pair_add_vec_kernel<TOut, 2>), 512);
+  else if (vec) NB_SPA((scaled_pair_add_vec_kernel<TOut, 4>), 512);
+  else NB_SPA(scaled_pair_add_kernel<TOut>, d >= 512 ? 256 : (d >= 128 ? 128 : 64));
+#undef NB_SPA
+  return 0;
+}
+
+NB_EXPORT int nb_scaled_pair_add(const float* a, float coef_a, const float* b, float coef_b, float* x,
+                                 const float* next_gamma, float next_eps, void* out_next,
+                                 int out_dtype, int n_rows, int d, cudaStream_t stream) {
+  if (n_rows == 0) return 0;
+  NB_REQUIRE(n_rows > 0 && d > 0 && (out_next == nullptr || next_gamma != nullptr) &&
+                 (out_next == nullptr || out_dtype == NB_F32 || out_dtype == NB_BF16),
+             NB_ERR_BAD_ARG, "scaled_pair_add: bad sizes rows=%d d=%d dtype=%d", n_rows, d, out_dtype);
+  const int rc = out_next == nullptr || out_dtype == NB_F32
+                     ? launch_scaled_pair_add<float>(a, coef_a, b, coef_b, x, next_gamma, next_eps,
+                                                     out_next, n_rows, d, stream)
+                     : launch_scaled_pair_add<__nv_bfloat16>(a, coef_a, b, coef_b, x, next_gamma,
+                                                             next_eps, out_next, n_rows, d, stream);
+  if (rc) return rc;
+  NB_CHECK_LAUNCH("scaled_pair_add");
   return 0;
 }
 

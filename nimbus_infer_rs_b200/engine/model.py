@@ -149,7 +149,7 @@ class Model:
                 x = self.stream_input.forward(ctx, x, x0)
                 ctx.normed = None
             ctx.kv, ctx.state, ctx.writes_cache = self.storage_of(ctx.cache, entry)
-            ctx.kv_extra = ctx.cache.layer_kv_extra(entry)
+            ctx.kv_extra = ctx.cache.layer_kv_extra(self.kv_source(entry))
             # an arrangement whose last pass over the stream can also norm it for the entry that
             # runs next is told that entry's first norm
             ctx.next_norm = ctx.next_block = None
@@ -166,7 +166,8 @@ class Model:
 
     def storage_requests(self):
         """What each schedule entry keeps per sequence: ``({entry: KVRequest}, {entry:
-        StateRequest})``.  An entry of a layer with ``cache_from`` keeps no keys/values."""
+        StateRequest})``.  An entry of a layer with ``cache_from`` keeps no keys/values; what it
+        sees is kept for it by the entry whose store it reads (the longer of the two windows)."""
         kv, st = {}, {}
         for entry, li in enumerate(self.run_order):
             layer = self.layers[li]
@@ -175,16 +176,15 @@ class Model:
                 if r is not None:
                     kv[entry] = r
             else:
-                # the reader must want what the owner keeps: same heads and head size, and no
-                # keys from before the owner's window
-                own = self.layers[layer.spec.cache_from].mixer.cache_request()
-                ok = (r is not None and own is not None and r.n_kv_heads == own.n_kv_heads
-                      and r.head_dim == own.head_dim
-                      and (own.window == 0 or 0 < r.window <= own.window))
-                if not ok:
-                    raise ValueError(
-                        f"layer {li} reads the cache of layer {layer.spec.cache_from}, which "
-                        f"keeps {own}, but asks for {r}")
+                # the reader must want what the owner keeps: same heads and sizes
+                src = self.kv_source(entry)
+                try:
+                    if r is None or src not in kv:
+                        raise ValueError(f"one keeps {kv.get(src)}, the other asks for {r}")
+                    kv[src] = kv[src].covering(r)
+                except ValueError as e:
+                    raise ValueError(f"layer {li} reads the cache of layer "
+                                     f"{layer.spec.cache_from}: {e}") from None
             s = layer.mixer.state_request()
             if s is not None:
                 st[entry] = s
@@ -197,8 +197,9 @@ class Model:
         """The further paged stores of each schedule entry's mixer: ``{(entry, k): KVRequest}``."""
         out = {}
         for entry, li in enumerate(self.run_order):
+            src = self.kv_source(entry)
             for k, r in enumerate(self.layers[li].mixer.extra_cache_requests()):
-                out[(entry, k)] = r
+                out[(src, k)] = out[(src, k)].covering(r) if src != entry else r
         return out
 
     def kv_source(self, entry: int) -> int:

@@ -5,3 +5,4 @@ from . import rizitar  # noqa: F401
 from . import pinozen  # noqa: F401
 from . import lulizen  # noqa: F401
 from . import bumulix  # noqa: F401
+from . import zorulix  # noqa: F401

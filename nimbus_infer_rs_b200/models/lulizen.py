@@ -133,18 +133,17 @@ def weight_plan(cfg: LulizenConfig, spec: ModelSpec, names: set[str]) -> WeightP
             if ff.shared is not None:
                 # the router's rows ride under the shared expert's gate and up halves
                 r[L + "ffn.shared.fc.weight"] = _gate_up(p + "mlp.shared.", ff.shared.ff, D,
-                                                         extra=(p + "mlp.router", E))
+                                                         extra=[(p + "mlp.router", E)])
                 r[L + "ffn.shared.proj.weight"] = take(p + "mlp.shared.down", (D, ff.shared.ff))
     return WeightPlan(r, ignored)
 
 
-def _gate_up(prefix: str, hidden: int, width: int, extra: tuple[str, int] | None = None) -> Recipe:
+def _gate_up(prefix: str, hidden: int, width: int, extra=()) -> Recipe:
     """Gate and up one under the other, each half filled with rows of zeros up to a multiple of
-    8 rows (the layout of ``gated_mlp``'s first product); ``extra`` = (name, rows): one more
-    matrix under them, filled up likewise."""
+    8 rows (the layout of ``gated_mlp``'s first product); ``extra`` = ((name, rows), ...): more
+    matrices under them, filled up likewise once all are there."""
     named = [(prefix + "gate", (hidden, width)), (prefix + "up", (hidden, width))]
-    if extra is not None:
-        named.append((extra[0], (extra[1], width)))
+    named += [(name, (rows, width)) for name, rows in extra]
     inner = _rows(named)
 
     def combine(ts):
@@ -152,7 +151,8 @@ def _gate_up(prefix: str, hidden: int, width: int, extra: tuple[str, int] | None
         if len(kinds) > 1:
             ts = [t.to(torch.float32) for t in ts]
         out = []
-        for t in ts:
+        blocks = list(ts[:2]) + ([torch.cat(list(ts[2:]), dim=0)] if len(ts) > 2 else [])
+        for t in blocks:
             out.append(t)
             pad = -t.shape[0] % 8
             if pad:

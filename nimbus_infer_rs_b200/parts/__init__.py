@@ -18,5 +18,6 @@ from .masked_attention import MaskedAttention
 from .differential_attention import DifferentialAttention
 from .selective_scan import SelectiveScan
 from .linear_attention import DecayedLinearAttention
-from .mixer_pair import NormedPair
+from .mixer_pair import NormedPair, ScaledPair
+from .gated_delta import GatedDeltaRule
 from .stream_input import EmbeddingRemix

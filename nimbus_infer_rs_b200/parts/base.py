@@ -19,8 +19,9 @@ family         interface
 ``block``      ``forward(ctx, x, layer)``: the arrangement of norms, mixer and feed-forward
                around the residual stream of one layer (``layer.ffn`` and ``layer.norm_ffn``
                are ``None`` in a layer without them)
-``side``       ``forward(ctx, x, x_act)``: a per-token input that a layer adds to the stream
-               after its sublayers (``x_act``: the stream's rows in the activation type)
+``side``       ``forward(ctx, x, x_act, then=None)``: a per-token input that a layer adds to
+               the stream after its sublayers (``x_act``: the stream's rows in the activation
+               type; ``then``: a norm whose rows of the new stream are returned)
 ``stream``     ``forward(ctx, x, x0) -> x'``: acts on the stream right before a schedule entry
                (``x0``: the embedding's output); the model lists which entries
 ``embedding``  ``forward(ctx, position) -> x``: the fp32 stream from the step's tokens; the
@@ -33,7 +34,7 @@ loaded device tensors through :meth:`Part.bind`.
 """
 from __future__ import annotations
 
-from dataclasses import dataclass, field
+from dataclasses import dataclass, field, replace
 from typing import Any, Callable
 
 import torch
@@ -69,13 +70,28 @@ class KVRequest:
     and value at once).  ``every`` > 1: one entry per ``every`` tokens of the sequence instead of
     one per token (a store of pooled blocks: entry ``b`` belongs to tokens ``b * every ..
     b * every + every - 1`` and exists once the last of them is cached).  ``keep_first`` (with a
-    window): the sequence's first ``keep_first`` tokens are read by every later token too."""
+    window): the sequence's first ``keep_first`` tokens are read by every later token too.
+    ``value_dim``: the size of a value where it is not the key's ``head_dim``."""
     n_kv_heads: int
     head_dim: int
     window: int = 0
     planes: int = 2
     every: int = 1
     keep_first: int = 0
+    value_dim: int | None = None
+
+    @property
+    def value_size(self) -> int:
+        return self.head_dim if self.value_dim is None else self.value_dim
+
+    def covering(self, other: "KVRequest") -> "KVRequest":
+        """This store kept for a second reader too: nothing that ``other`` sees is given back.
+        Both ask for heads and sizes of one kind."""
+        if (self.n_kv_heads, self.head_dim, self.value_size, self.planes, self.every) != (
+                other.n_kv_heads, other.head_dim, other.value_size, other.planes, other.every):
+            raise ValueError(f"one keeps {self}, the other asks for {other}")
+        window = max(self.window, other.window) if self.window and other.window else 0
+        return replace(self, window=window, keep_first=max(self.keep_first, other.keep_first))
 
 
 @dataclass(frozen=True)
@@ -189,7 +205,7 @@ class FeedForward(Part):
 class Side(Part):
     family = "side"
 
-    def forward(self, ctx, x: torch.Tensor, x_act: torch.Tensor) -> None:
+    def forward(self, ctx, x: torch.Tensor, x_act: torch.Tensor, then: "Norm | None" = None):
         raise NotImplementedError
 
 

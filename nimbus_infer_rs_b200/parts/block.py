@@ -11,28 +11,53 @@ from .norm import RMSNorm
 class PreNormBlock(Block):
     """``x += mixer(norm_mixer(x)); x += ffn(norm_ffn(x))`` (src/model.rs:297-300 with
     :345-357, :437-439, :448-460, :485-487).  ``x`` is the fp32 residual stream.  The
-    feed-forward may be absent (then the layer is its first half).  A mixer that adds its result
+    feed-forward may be absent.  A mixer that adds its result
     in a row pass of its own (``takes_next_norm``) is given the feed-forward's norm and hands
-    back that norm's rows, computed in the same pass."""
+    back that norm's rows, computed in the same pass.
+
+    A per-token input (``layer.side``) comes last.  It multiplies the stream by a matrix, so it
+    wants the stream's rows in the activation type, which a feed-forward whose last kernel is a
+    row pass (``hands_out_rounded``) leaves beside its addition; and its own pass over the stream
+    also norms it for the layer that runs next (``ctx.next_norm``, ``ctx.normed``)."""
     graph_safe = True
+    takes_handed_norm = True
 
     def __init__(self):
         pass
 
     def forward(self, ctx, x, layer) -> None:
-        mixer, ffn = layer.mixer, layer.ffn
-        h = layer.norm_mixer.defer(ctx, x) if mixer.accepts_deferred_norm \
-            else layer.norm_mixer.forward(ctx, x)
-        if ffn is None:
-            mixer.forward(ctx, h, x)
-            return
-        if getattr(mixer, "takes_next_norm", False) and hasattr(layer.norm_ffn, "add_into"):
-            h = mixer.forward(ctx, h, x, then=layer.norm_ffn)
+        mixer, ffn, side = layer.mixer, layer.ffn, layer.side
+        h, ctx.normed = ctx.normed, None
+        if h is None:
+            h = layer.norm_mixer.defer(ctx, x) if mixer.accepts_deferred_norm \
+                else layer.norm_mixer.forward(ctx, x)
+        rounded = x if side is None or ctx.rt.act_dtype == torch.float32 else None
+        if ffn is not None:
+            h = self._mix(ctx, h, x, layer)
+            if rounded is None and getattr(ffn, "hands_out_rounded", False):
+                rounded = torch.empty(x.shape, device=x.device, dtype=ctx.rt.act_dtype)
+                ffn.forward(ctx, h, x, rounded=rounded)
+            else:
+                ffn.forward(ctx, h, x)
         else:
             mixer.forward(ctx, h, x)
-            h = layer.norm_ffn.defer(ctx, x) if ffn.accepts_deferred_norm \
-                else layer.norm_ffn.forward(ctx, x)
-        ffn.forward(ctx, h, x)
+        if side is None:
+            return
+        if rounded is None:
+            rounded = torch.empty(x.shape, device=x.device, dtype=ctx.rt.act_dtype)
+            ctx.ops.cast_cols(x, rounded, 0)
+        then = ctx.next_norm if isinstance(ctx.next_norm, RMSNorm) else None
+        ctx.normed = side.forward(ctx, x, rounded, then)
+
+    @staticmethod
+    def _mix(ctx, h, x, layer):
+        """The mixer's result into the stream; returns the feed-forward's normed rows."""
+        mixer, ffn = layer.mixer, layer.ffn
+        if getattr(mixer, "takes_next_norm", False) and hasattr(layer.norm_ffn, "add_into"):
+            return mixer.forward(ctx, h, x, then=layer.norm_ffn)
+        mixer.forward(ctx, h, x)
+        return layer.norm_ffn.defer(ctx, x) if ffn.accepts_deferred_norm \
+            else layer.norm_ffn.forward(ctx, x)
 
 
 @register_part("block", "parallel")

@@ -66,12 +66,14 @@ class GatedMLP(FeedForward):
 
     ``extra_outputs`` > 0: that many more rows of weights ride on the first product for another
     reader of the same rows (a router beside a shared expert); their fp32 results are left in
-    ``ctx.shared_projection`` as ``(rows, first column)``."""
+    ``ctx.shared_projection`` as ``(rows, first column)``.  ``row_gate``: one more weight row behind
+    those, whose result ``z`` multiplies the whole row's output by ``sigmoid(z)`` (in fp32, in the
+    pass between the two products)."""
     graph_safe = True
     can_overwrite = True
 
     def __init__(self, width: int, hidden: int, activation: str, limit: float | None = None,
-                 extra_outputs: int = 0):
+                 extra_outputs: int = 0, row_gate: bool = False):
         if activation not in GLU_ACTIVATIONS:
             raise ValueError(f"unknown activation {activation!r} (have {sorted(GLU_ACTIVATIONS)})")
         if (limit is not None) != (activation in PARAM_ACTIVATIONS):
@@ -83,7 +85,9 @@ class GatedMLP(FeedForward):
         # the two halves start on multiples of 8 columns (fp32 rows on 32-byte boundaries)
         self.half = -(-self.hidden // 8) * 8
         self.extra_outputs = int(extra_outputs)
-        self.fc = Linear(self.width, 2 * self.half + -(-self.extra_outputs // 8) * 8, bias=False)
+        more = self.extra_outputs + (1 if row_gate else 0)
+        self.col_row_gate = 2 * self.half + self.extra_outputs if row_gate else -1
+        self.fc = Linear(self.width, 2 * self.half + -(-more // 8) * 8, bias=False)
         self.proj = Linear(self.hidden, self.width, bias=False)
 
     def children(self):
@@ -94,7 +98,7 @@ class GatedMLP(FeedForward):
         if self.extra_outputs:
             ctx.shared_projection = (both, 2 * self.half)
         mid = torch.empty((both.shape[0], self.hidden), device=both.device, dtype=ctx.rt.act_dtype)
-        ctx.ops.glu_rows(both, 0, self.half, self.act_code, mid, self.act_param)
+        ctx.ops.glu_rows(both, 0, self.half, self.act_code, mid, self.act_param, self.col_row_gate)
         if accumulate:
             self.proj(ctx, mid, residual=residual)
         else:

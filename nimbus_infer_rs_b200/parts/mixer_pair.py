@@ -1,4 +1,4 @@
-"""Two mixers side by side on the same input, their normed results averaged."""
+"""Two mixers side by side on the same input, their results combined in one pass over the stream."""
 from __future__ import annotations
 
 import torch
@@ -6,27 +6,24 @@ import torch
 from .base import VECTOR, Mixer, ParamSpec, PartSpec, StateRequest, build_part, register_part
 
 
-@register_part("mixer", "normed_pair")
-class NormedPair(Mixer):
-    """``left`` and ``right`` (any two mixers, given as part descriptions) read the same rows;
-    each result is RMS-normed over the width with a weight of its own (``left_norm``,
-    ``right_norm``; a plain weight) and the pair's result is ``coef`` times their sum.
+class MixerPair(Mixer):
+    """``left`` and ``right`` (any two mixers, given as part descriptions) read the same rows and
+    write into fp32 buffers of their own; ``combine`` (a subclass's) adds the two to the stream
+    in one row pass that also hands out, when the arrangement asks for it, the normed rows of the
+    stream's next reader.
 
-    Each branch writes into an fp32 buffer of its own; one row pass norms both, adds the
-    average to the stream and, when the arrangement asks for it, hands out the normed rows of
-    the stream's next reader.  Storage: the pair asks for what its branches ask for, the paged
-    stores one after the other and the fixed-size state side by side in one row (the left
-    branch's numbers first); each branch sees its own part.
+    Storage: the pair asks for what its branches ask for, the paged stores one after the other
+    and the fixed-size state side by side in one row (the left branch's numbers first); each
+    branch sees its own part.
     """
     can_overwrite = False
     takes_next_norm = True       # `forward(..., then=norm)` returns that norm's rows of the stream
 
-    def __init__(self, width: int, eps: float, left: PartSpec, right: PartSpec, coef: float = 0.5):
-        self.width, self.eps, self.coef = int(width), float(eps), float(coef)
+    def __init__(self, width: int, left: PartSpec, right: PartSpec):
+        self.width = int(width)
         self.left = build_part("mixer", left)
         self.right = build_part("mixer", right)
         self.graph_safe = bool(self.left.graph_safe and self.right.graph_safe)
-        self.left_norm = self.right_norm = None
         # paged stores: every branch's own first, then its further ones, in the order asked
         self._stores = []           # (branch index, is_main)
         for b, part in enumerate((self.left, self.right)):
@@ -39,10 +36,6 @@ class NormedPair(Mixer):
 
     def children(self):
         return {"left": self.left, "right": self.right}
-
-    def param_specs(self):
-        return {"left_norm": ParamSpec((self.width,), VECTOR),
-                "right_norm": ParamSpec((self.width,), VECTOR)}
 
     def cache_request(self):
         return self._stores[0][2] if self._stores else None
@@ -74,6 +67,11 @@ class NormedPair(Mixer):
             ctx.kv, ctx.kv_extra, ctx.state, ctx.writes_cache = kv, extra, state, writes
         return y
 
+    def combine(self, ctx, a, b, residual, norm_args) -> None:
+        """Add the branches' results to the stream; ``norm_args``: the next reader's norm weight,
+        its eps and the rows to fill (or three times nothing)."""
+        raise NotImplementedError
+
     def forward(self, ctx, h: torch.Tensor, residual: torch.Tensor, then=None):
         """``then``: the norm in front of the stream's next reader; its rows are returned."""
         a = self._branch(ctx, 0, self.left, h, residual)
@@ -81,7 +79,38 @@ class NormedPair(Mixer):
         nxt = None
         if then is not None:
             nxt = torch.empty(residual.shape, device=residual.device, dtype=ctx.rt.act_dtype)
-        ctx.ops.rms_pair_add(a, self.left_norm, b, self.right_norm, self.eps, self.coef, residual,
-                             then.weight if then is not None else None,
-                             then.eps if then is not None else 0.0, nxt)
+        self.combine(ctx, a, b, residual, (then.weight, then.eps, nxt) if then is not None
+                     else (None, 0.0, None))
         return nxt
+
+
+@register_part("mixer", "normed_pair")
+class NormedPair(MixerPair):
+    """Each result is RMS-normed over the width with a weight of its own (``left_norm``,
+    ``right_norm``; a plain weight) and the pair's result is ``coef`` times their sum."""
+
+    def __init__(self, width: int, eps: float, left: PartSpec, right: PartSpec, coef: float = 0.5):
+        super().__init__(width, left, right)
+        self.eps, self.coef = float(eps), float(coef)
+        self.left_norm = self.right_norm = None
+
+    def param_specs(self):
+        return {"left_norm": ParamSpec((self.width,), VECTOR),
+                "right_norm": ParamSpec((self.width,), VECTOR)}
+
+    def combine(self, ctx, a, b, residual, norm_args) -> None:
+        ctx.ops.rms_pair_add(a, self.left_norm, b, self.right_norm, self.eps, self.coef, residual,
+                             *norm_args)
+
+
+@register_part("mixer", "scaled_pair")
+class ScaledPair(MixerPair):
+    """The pair's result is ``left_scale * left + right_scale * right`` (constants)."""
+
+    def __init__(self, width: int, left: PartSpec, right: PartSpec, left_scale: float = 1.0,
+                 right_scale: float = 1.0):
+        super().__init__(width, left, right)
+        self.left_scale, self.right_scale = float(left_scale), float(right_scale)
+
+    def combine(self, ctx, a, b, residual, norm_args) -> None:
+        ctx.ops.scaled_pair_add(a, self.left_scale, b, self.right_scale, residual, *norm_args)

@@ -145,8 +145,15 @@ class CpuBackend:
                 self._entry(kv, kv.v, slot, pos)[:] = k.to(kv.v.dtype)
 
     def qkv_norm_rope_append(self, src, q_col, k_col, v_col, q_gamma, k_gamma, eps, freq, rot_dims,
-                             amplitude, layout, k_store, v_store, n_heads, value_dim, q_out, write):
+                             amplitude, layout, k_store, v_store, n_heads, value_dim, q_out, write,
+                             whole=False):
         d, G = k_store.head_dim, k_store.n_kv_heads
+
+        def normed(x, gamma):
+            over = (0, 1) if whole else -1
+            gamma = gamma.view(x.shape) if whole else gamma
+            return x / torch.sqrt((x * x).mean(over, keepdim=True) + eps) * gamma
+
         half = rot_dims // 2
 
         def turn(x, pos):
@@ -164,12 +171,13 @@ class CpuBackend:
                 continue
             pos = int(layout.row_pos[r])
             q = src[r, q_col:q_col + n_heads * d].float().view(n_heads, d)
-            k = src[r, k_col:k_col + G * d].float().view(G, d)
             if q_gamma is not None:
-                q = q / torch.sqrt((q * q).mean(-1, keepdim=True) + eps) * q_gamma
-                k = k / torch.sqrt((k * k).mean(-1, keepdim=True) + eps) * k_gamma
+                q = normed(q, q_gamma)
             q_out[r] = turn(q, pos).reshape(-1).to(q_out.dtype)
             if write:
+                k = src[r, k_col:k_col + G * d].float().view(G, d)
+                if k_gamma is not None:
+                    k = normed(k, k_gamma)
                 self._entry(k_store, k_store.k, slot, pos)[:] = turn(k, pos).to(k_store.k.dtype)
                 vals = self._values_of(k_store, v_store)
                 v = src[r, v_col:v_col + G * value_dim].float().view(G, value_dim)
@@ -177,7 +185,8 @@ class CpuBackend:
 
     def attention_masked(self, q, layout, k_store, v_store, n_heads, sink, out, scale, softcap=0.0,
                          window=0, keep_first=0, chunk=0, gate=None, gate_col=0):
-        d, dv, G = k_store.head_dim, v_store.head_dim, k_store.n_kv_heads
+        d, G = k_store.head_dim, k_store.n_kv_heads
+        dv = v_store.value_size if v_store is k_store else v_store.head_dim
         group = n_heads // G
         for r in range(layout.n_rows):
             slot = int(layout.row_slot[r])
@@ -305,6 +314,34 @@ class CpuBackend:
             o = torch.einsum("hkv,hk->hv", S, rr)
             o = o / torch.sqrt((o * o).mean(-1, keepdim=True) + eps)
             out[r] = (o.reshape(hd) * norm_w * g).to(out.dtype)
+
+    def gated_delta(self, qkv, beta, col_beta, low, col_decay, col_gate, a_log, dt_bias, norm, eps,
+                    key_eps, layout, state, n_heads, n_kv_heads, d, dv, out):
+        H, G = n_heads, n_kv_heads
+        of = torch.arange(H) // (H // G)
+        for r in range(layout.n_rows):
+            slot = int(layout.row_slot[r])
+            if slot < 0:
+                out[r].zero_()
+                continue
+            row = qkv[r].float()
+
+            def unit(x):
+                return x / torch.sqrt((x * x).sum(-1, keepdim=True) + key_eps)
+            q = unit(row[:G * d].view(G, d))[of] * d ** -0.5
+            k = unit(row[G * d:2 * G * d].view(G, d))[of]
+            v = row[2 * G * d:2 * G * d + H * dv].view(H, dv)
+            rate = torch.sigmoid(beta[r, col_beta:col_beta + H].float())
+            dt = torch.nn.functional.softplus(low[r, col_decay:col_decay + H * d] + dt_bias).view(H, d)
+            g = torch.exp(-torch.exp(a_log)[:, None] * dt)
+            S = state[slot].view(H, d, dv)
+            S *= g[:, :, None]
+            u = rate[:, None] * (v - torch.einsum("hkv,hk->hv", S, k))
+            S += k[:, :, None] * u[:, None, :]
+            o = torch.einsum("hkv,hk->hv", S, q)
+            o = o / torch.sqrt((o * o).mean(-1, keepdim=True) + eps) * norm
+            gate = torch.sigmoid(low[r, col_gate:col_gate + H * dv])
+            out[r] = (o.reshape(-1) * gate).to(out.dtype)
 
     # -- short convolutions, capped attention, linear recurrences (row by row, in order) ---
     @staticmethod
@@ -454,6 +491,13 @@ class CpuBackend:
             u = residual / torch.sqrt((residual * residual).mean(-1, keepdim=True) + next_eps)
             out_next.copy_((u * next_gamma).to(out_next.dtype))
 
+    def scaled_pair_add(self, a, scale_a, b, scale_b, residual, next_gamma=None, next_eps=0.0,
+                        out_next=None):
+        residual += scale_a * a.float() + scale_b * b.float()
+        if out_next is not None:
+            u = residual / torch.sqrt((residual * residual).mean(-1, keepdim=True) + next_eps)
+            out_next.copy_((u * next_gamma).to(out_next.dtype))
+
     @classmethod
     def _gate_up(cls, gate, up, act, param):
         if act == 8:
@@ -461,10 +505,13 @@ class CpuBackend:
             return g * torch.sigmoid(1.702 * g) * (torch.clamp(up, -param, param) + 1.0)
         return cls._act(gate, act) * up
 
-    def glu_rows(self, x, gate_col, up_col, act, out, act_param=0.0):
+    def glu_rows(self, x, gate_col, up_col, act, out, act_param=0.0, row_gate_col=-1):
         n, d = out.shape
-        out.copy_(self._gate_up(x[:n, gate_col:gate_col + d].float(),
-                                x[:n, up_col:up_col + d].float(), act, act_param).to(out.dtype))
+        y = self._gate_up(x[:n, gate_col:gate_col + d].float(), x[:n, up_col:up_col + d].float(),
+                          act, act_param)
+        if row_gate_col >= 0:
+            y = y * torch.sigmoid(x[:n, row_gate_col:row_gate_col + 1].float())
+        out.copy_(y.to(out.dtype))
 
     def cast_cols(self, x, out, out_col):
         out[:, out_col:out_col + x.shape[1]] = x.to(out.dtype)
@@ -546,9 +593,10 @@ class CpuBackend:
                 den = den + torch.exp(sink - m)
             out[r] = ((e / den[:, None]) @ c[:, :dv]).reshape(-1).to(out.dtype)
 
-    def moe_route(self, logits, col, n_experts, top, renormalize, layout, idx, weight):
+    def moe_route(self, logits, col, n_experts, top, renormalize, layout, idx, weight, bias=None):
         n = layout.n_rows
-        s = torch.softmax(logits[:n, col:col + n_experts].float(), dim=-1)
+        z = logits[:n, col:col + n_experts].float()
+        s = torch.softmax(z if bias is None else z + bias, dim=-1)
         order = torch.sort(s, dim=-1, descending=True, stable=True).indices[:, :top]
         w = torch.gather(s, 1, order)
         if renormalize:
@@ -611,7 +659,7 @@ class CpuBackend:
                     v = v * (w2[e].float() @ x[row].float())
                 out[at] = v.to(out.dtype)
 
-    def moe_combine(self, y, place, weight, residual):
+    def moe_combine(self, y, place, weight, residual, out_cast=None):
         n, top = weight.shape
         pl = place.reshape(-1)
         for r in range(n):
@@ -619,6 +667,8 @@ class CpuBackend:
                 at = int(pl[r * top + k])
                 if at >= 0:
                     residual[r] += weight[r, k] * y[at]
+        if out_cast is not None:
+            out_cast.copy_(residual.to(out_cast.dtype))
 
     def linear(self, x, w, bias, out, act=0, residual=None, norm=None):
         if norm is not None:

@@ -257,5 +257,12 @@ def test_a_reader_must_want_what_the_owner_keeps():
                        norm_ffn=bad[3].norm_ffn, cache_from=1)
     m = Model(ModelSpec("toy_mixed_lm", 131, 48, 256, spec.position, tuple(bad), spec.final_norm),
               Runtime(torch.device("cpu"), torch.float32))
+    # a wider window: the owner's store keeps what the reader sees
+    assert m.storage_requests()[0][1].window == 90
+    other = PartSpec("causal_attention", {**spec.layers[3].mixer.args, "head_dim": 16})
+    bad[3] = LayerSpec(mixer=other, ffn=bad[3].ffn, norm_mixer=bad[3].norm_mixer,
+                       norm_ffn=bad[3].norm_ffn, cache_from=1)
+    m = Model(ModelSpec("toy_mixed_lm", 131, 48, 256, spec.position, tuple(bad), spec.final_norm),
+              Runtime(torch.device("cpu"), torch.float32))
     with pytest.raises(ValueError, match="reads the cache of layer 1"):
         m.storage_requests()

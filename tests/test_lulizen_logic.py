@@ -189,12 +189,12 @@ def test_storage_per_run_and_what_each_mask_keeps(models, cpu_backend):
     e = _engine(models, "A")
     kv, st = e.model.storage_requests()
     extra = e.model.extra_storage_requests()
-    # four runs; run 0 keeps keys and (wider) values in a store each; runs 1 and 2 share tensors
-    # and keep a store each; the embedding keeps the token before
-    assert sorted(kv) == [0, 1, 2, 3] and sorted(extra) == [(0, 0)]
+    # four runs; run 0 keeps keys and (wider) values in a store; runs 1 and 2 share tensors and
+    # keep a store each; the embedding keeps the token before
+    assert sorted(kv) == [0, 1, 2, 3] and not extra
     assert sorted(st) == [-1] and st[-1].n_elements == 1
-    assert kv[0] == KVRequest(2, 12, 9, planes=1, keep_first=3)
-    assert extra[(0, 0)] == KVRequest(2, 20, 9, planes=1, keep_first=3)
+    assert kv[0] == KVRequest(2, 12, 9, keep_first=3, value_dim=20)
+    assert e.cache.layer_kv(0).k.shape[1:] == (2, 64, 12) and e.cache.layer_kv(0).v.shape[1:] == (2, 64, 20)
     assert kv[1] == kv[2] == KVRequest(3, 16, 11, planes=2)
     assert e.cache.layer_kv(1).k.data_ptr() != e.cache.layer_kv(2).k.data_ptr()
     assert kv[3] == KVRequest(1, 24, 40, planes=2)
