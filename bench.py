@@ -300,7 +300,11 @@ DESIGN_PAIRS = {"runesun": (("runesun-2k", "gpt2-2k"), ("runesun-1k", "gpt2-1k")
                 # beside the two closest designs: Lulizen's masked attention over shared key heads
                 # and Runesun's attention over a latent
                 "bumulix": (("bumulix-2k", "lulizen-2k", "runesun-2k"),
-                            ("bumulix-1k", "lulizen-1k", "runesun-1k"))}
+                            ("bumulix-1k", "lulizen-1k", "runesun-1k")),
+                # beside the two closest designs: Lulizen's masked attention and routed experts
+                # with a shared one, Rizitar's delta rule and per-token input
+                "zorulix": (("zorulix-2k", "lulizen-2k", "rizitar-2k"),
+                            ("zorulix-1k", "lulizen-1k", "rizitar-1k"))}
 
 
 class OpTimer:
@@ -315,7 +319,7 @@ class OpTimer:
              "selective_scan", "linear_attention", "rmsnorm_gated", "rms_pair_add", "glu_rows",
              "cast_cols", "embed_hashed", "ln_add", "qkv_norm_rope_append",
              "attention_masked", "moe_route_sigmoid", "attention_differential",
-             "latent_rope_append", "streams", "softcap_rows")
+             "latent_rope_append", "streams", "softcap_rows", "gated_delta", "scaled_pair_add")
 
     def __init__(self, ops):
         import torch
@@ -362,7 +366,13 @@ class OpTimer:
         if kind == "moe_linear":
             return "moe_linear gate+up" if a[5] is not None else (
                 "moe_linear up" if a[1] is not None else "moe_linear down")
+        if kind == "attention_masked" and self._value_size(a[2], a[3]) != a[2].head_dim:
+            return f"attention_masked, keys of {a[2].head_dim}, values of {self._value_size(a[2], a[3])}"
         return kind
+
+    @staticmethod
+    def _value_size(keys, values):
+        return keys.value_size if values is keys else values.head_dim
 
     def _work(self, kind, a, kw):
         """(bytes, flops) of one call."""
@@ -401,7 +411,16 @@ class OpTimer:
             out = a[4] if kind == "layernorm" else a[3]
             return 4 * out.numel() + nb(out), 0
         if kind == "moe_combine":
-            return nb(a[0]) + 2 * nb(a[3]), 0
+            return nb(a[0], a[4] if len(a) > 4 else None) + 2 * nb(a[3]), 0
+        if kind == "scaled_pair_add":
+            return nb(a[0], a[2], a[7]) + 2 * nb(a[4]), 0
+        if kind == "gated_delta":
+            lay, heads, kv_heads, d, dv, out = a[11], a[13], a[14], a[15], a[16], a[17]
+            # convolved q, k, v, the logits of rate, decay and gate per token, the state of every
+            # sequence in and out; per token and head 4 d dv multiply-adds on the CUDA cores
+            per_token = 2 * kv_heads * d + heads * (2 * dv + d + 1)
+            return lay.n_tokens * per_token * 4 + nb(out) + 2 * lay.n_seqs * heads * d * dv * 4, \
+                2 * 4 * lay.n_tokens * heads * d * dv
         if kind in ("rms_add", "ln_add"):
             return nb(a[0], a[6], a[7]) + 2 * nb(a[3]), 0
         if kind == "embed_hashed":
@@ -410,7 +429,7 @@ class OpTimer:
             return nb(a[0]) + 2 * nb(a[12]), 0
         if kind == "qkv_norm_rope_append":
             lay, ks, vs, heads, q = a[10], a[11], a[12], a[13], a[15]
-            kv = ks.n_kv_heads * (ks.head_dim + vs.head_dim)
+            kv = ks.n_kv_heads * (ks.head_dim + self._value_size(ks, vs)) if a[16] else 0
             return lay.n_tokens * (4 * (heads * ks.head_dim + kv) + kv * ks.k.element_size()) + nb(q), 0
         if kind == "attention_masked":
             q, lay, ks, vs, heads, out = a[0], a[1], a[2], a[3], a[4], a[6]
@@ -425,8 +444,8 @@ class OpTimer:
             # every sequence's keys once (neighbouring rows share them), queries, outputs
             keys = sum(p + n - first(p) + (min(keep, first(p)) if window else 0)
                        for p, n in zip(lay.seq_pos0_host, lay.seq_lens))
-            return keys * ks.n_kv_heads * (ks.head_dim + vs.head_dim) * elt + nb(q, out), \
-                2 * pairs * heads * (ks.head_dim + vs.head_dim)
+            both = ks.head_dim + self._value_size(ks, vs)
+            return keys * ks.n_kv_heads * both * elt + nb(q, out), 2 * pairs * heads * both
         if kind == "attention_differential":
             q, lay, ks, vs, heads, out, window = a[0], a[1], a[2], a[3], a[4], a[5], a[7]
 

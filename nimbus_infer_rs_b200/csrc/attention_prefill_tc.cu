@@ -1,6 +1,6 @@
 // Prefill attention on the 5th-generation tensor cores (sm_100a): many query rows per
-// sequence over the paged key/value cache, head size 64 or 128, bf16 operands, fp32 scores and
-// softmax.
+// sequence over the paged key/value cache, head size 64 or 128 (or, as a variant, keys and values
+// of different sizes up to 128), bf16 operands, fp32 scores and softmax.
 //
 // One CTA takes 128 consecutive query rows of one sequence and one head; a row of the tile is
 // a lane of tensor memory.  Warp 0 is the producer: one thread brings the query tile and then,
@@ -73,27 +73,32 @@ __device__ __forceinline__ void tc05_wait_st() {
   asm volatile("tcgen05.wait::st.sync.aligned;\n" ::: "memory");
 }
 
-template <int HD>
+// HK, HV: the sizes of a key and of a value, each 64 or 128 (as staged: see VAR below)
+template <int HK, int HV>
 struct AttnSmem {
-  static constexpr int HB = HD / 64;                      // 64-column boxes per row of a head
-  static constexpr int Q_BYTES = TILE_Q * 128 * HB;       // [HB][128 rows][128 B]
+  static constexpr int KB = HK / 64, VB = HV / 64;        // 64-column boxes per row of a key, a value
+  static constexpr int Q_BYTES = TILE_Q * 128 * KB;       // [KB][128 rows][128 B]
   static constexpr int PAGE_BOX = PAGE_TOKENS * 128;      // one page, 64 head columns: 8 KB
-  static constexpr int K_BYTES = 2 * PAGE_BOX * HB;       // [HB][2 pages][64 keys][128 B]
-  static constexpr int V_BYTES = K_BYTES;
+  static constexpr int K_BYTES = 2 * PAGE_BOX * KB;       // [KB][2 pages][64 keys][128 B]
+  static constexpr int V_BYTES = 2 * PAGE_BOX * VB;
   static constexpr int STAGE_BYTES = K_BYTES + V_BYTES;
-  static constexpr int STAGES = HD == 64 ? 4 : 2;         // 144 KB / 160 KB of tiles
+  static constexpr int STAGES = HK + HV == 128 ? 4 : HK + HV == 192 ? 3 : 2;   // 144 to 176 KB of tiles
   static constexpr int TILES_BYTES = Q_BYTES + STAGES * STAGE_BYTES;
   // q_full, kv_full[S], kv_empty[S], s_full[2], p_full[2], o_full[2], o_empty[2]
   static constexpr int N_BARRIERS = 1 + 2 * STAGES + 8;
   static constexpr int XCH_BYTES = 6 * TILE_Q * 4;   // row maxima (two buffers) and sums of the two halves
   static constexpr int TOTAL = TILES_BYTES + N_BARRIERS * 8 + 16 + XCH_BYTES + 1024 /* alignment slack */;
   // tensor memory columns: two score buffers of 128 (the probabilities of a turn take the
-  // first 64 columns of its score buffer), two output buffers of HD
+  // first 64 columns of its score buffer), two output buffers of HV
   static constexpr int S_COL = 0, O_COL = 256;
   static constexpr int TMEM_COLS = 512;
 };
 
-template <int HD, typename TOut, bool CAP>
+// VAR: keys of dk <= HK and values of dv <= HV numbers (multiples of 8): the tensor maps of the
+// cache end at dk and dv columns, so what a box holds beyond them is zeros (a query's box then
+// holds numbers of the next head there, which meet the key's zeros); no append.  Without VAR the
+// two sizes are HK and HV.
+template <int HK, int HV, typename TOut, bool CAP, bool VAR>
 __global__ void __launch_bounds__(TC_THREADS, 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                             const __grid_constant__ CUtensorMap map_k,
@@ -106,9 +111,10 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                             int out_stride, float scale, float softcap,
                             const float* __restrict__ sink, NbAttnOpts opt, int max_splits,
                             int chunk_pages, float* part, int* counters,
-                            int* err_word) {
-  using L = AttnSmem<HD>;
-  constexpr int HB = L::HB;
+                            int* err_word, int dk_given, int dv_given) {
+  using L = AttnSmem<HK, HV>;
+  constexpr int KB = L::KB, VB = L::VB;
+  const int dk = VAR ? dk_given : HK, dv = VAR ? dv_given : HV;
   extern __shared__ unsigned char smem_dyn[];
   const uint32_t raw = smem_u32(smem_dyn);
   const uint32_t base = (raw + 1023u) & ~1023u;
@@ -214,24 +220,24 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
     if (lane == 0) {   // ------------------------------------------------------ TMA producer
       mbar_expect_tx(q_full, L::Q_BYTES);
 #pragma unroll
-      for (int b = 0; b < HB; ++b)
-        tma_load_2d(q_smem + b * (TILE_Q * 128), &map_q, q_col + h * HD + b * 64, row0 + q0, q_full);
+      for (int b = 0; b < KB; ++b)
+        tma_load_2d(q_smem + b * (TILE_Q * 128), &map_q, q_col + h * dk + b * 64, row0 + q0, q_full);
       bool ok = true;
       // keys and values of page p of the sequence, 64 head columns at a time: from the cache,
       // or (append) from the step's own rows when the page lies at or after the cached length
       auto load_page = [&](int p, int page_id, uint32_t kb, uint32_t vb, int b, uint32_t bar) {
-        if (append && p * PAGE_TOKENS >= pos0) {
+        if (!VAR && append && p * PAGE_TOKENS >= pos0) {
           const int row = row0 + p * PAGE_TOKENS - pos0;
-          tma_load_2d(kb, &map_new, k_col + kvh * HD + b * 64, row, bar);
-          tma_load_2d(vb, &map_new, v_col + kvh * HD + b * 64, row, bar);
+          tma_load_2d(kb, &map_new, k_col + kvh * HK + b * 64, row, bar);
+          tma_load_2d(vb, &map_new, v_col + kvh * HV + b * 64, row, bar);
         } else {
           const int row = (page_id * n_kv_heads + kvh) * PAGE_TOKENS;
-          tma_load_2d(kb, &map_k, b * 64, row, bar);
-          tma_load_2d(vb, &map_v, b * 64, row, bar);
+          if (KB == VB || b < KB) tma_load_2d(kb, &map_k, b * 64, row, bar);
+          if (KB == VB || b < VB) tma_load_2d(vb, &map_v, b * 64, row, bar);
         }
       };
       // (append) a page of this tile's own query rows goes from shared memory into the cache
-      const bool writer = append && (h % group == 0);
+      const bool writer = !VAR && append && (h % group == 0);
       bool stored = false;
       auto store_page = [&](int p, int page_id, uint32_t kb, uint32_t vb, int b) {
         if (p * PAGE_TOKENS < pos0 + q0) return;
@@ -256,7 +262,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
         const uint32_t k_dst = kv_smem + st * L::STAGE_BYTES;
         const int pa = p_begin + 2 * j;
 #pragma unroll
-        for (int b = 0; b < HB; ++b) {
+        for (int b = 0; b < (KB > VB ? KB : VB); ++b) {
           const uint32_t kb = k_dst + b * (2 * L::PAGE_BOX), vb = kb + L::K_BYTES;
           load_page(pa, page_a, kb, vb, b, kv_full(st));
           if (two) load_page(pa + 1, page_b, kb + L::PAGE_BOX, vb + L::PAGE_BOX, b, kv_full(st));
@@ -266,7 +272,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
           ok = mbar_wait(kv_full(st), (j / L::STAGES) & 1u, abort_flag);
           if (!ok) break;
 #pragma unroll
-          for (int b = 0; b < HB; ++b) {
+          for (int b = 0; b < KB; ++b) {
             const uint32_t kb = k_dst + b * (2 * L::PAGE_BOX), vb = kb + L::K_BYTES;
             store_page(pa, page_a, kb, vb, b);
             if (two) store_page(pa + 1, page_b, kb + L::PAGE_BOX, vb + L::PAGE_BOX, b);
@@ -281,7 +287,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
     if (lane == 0) {   // ------------------------------------------------------ MMA issuer
       constexpr uint32_t idesc_s2 = instr_desc_bf16(TILE_Q, 2 * PAGE_TOKENS);   // two pages of keys
       constexpr uint32_t idesc_s1 = instr_desc_bf16(TILE_Q, PAGE_TOKENS);       // one
-      constexpr uint32_t idesc_o = instr_desc_bf16_b_mn(TILE_Q, HD);
+      constexpr uint32_t idesc_o = instr_desc_bf16_b_mn(TILE_Q, HV);
       bool ok = mbar_wait(q_full, 0u, abort_flag);
       tc05_fence_after();
       // O_i = P_i V_i: A = the probabilities in tensor memory (16 keys = 8 columns per MMA),
@@ -296,7 +302,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
         tc05_fence_after();
         const uint32_t v_addr = kv_smem + st * L::STAGE_BYTES + L::K_BYTES;
         const uint32_t a_tmem = tmem_base + L::S_COL + b * (2 * PAGE_TOKENS);
-        const uint32_t d_tmem = tmem_base + L::O_COL + b * HD;
+        const uint32_t d_tmem = tmem_base + L::O_COL + b * HV;
         const int k_steps = two_pages(i) ? 8 : 4;
 #pragma unroll
         for (int k = 0; k < 8; ++k) {
@@ -319,7 +325,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
         const uint32_t d_tmem = tmem_base + L::S_COL + b * (2 * PAGE_TOKENS);
         const uint32_t idesc_s = two_pages(j) ? idesc_s2 : idesc_s1;
 #pragma unroll
-        for (int k = 0; k < HD / 16; ++k) {
+        for (int k = 0; k < HK / 16; ++k) {
+          if (VAR && k * 16 >= dk) break;
           // 16 head columns per MMA: 32 bytes inside a 64-column box, the next box after four
           const uint32_t box = k >> 2, in_box = (k & 3) * 2;
           const uint64_t da = smem_desc_sw128(q_smem + box * (TILE_Q * 128)) + in_box;
@@ -346,7 +353,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
     // scores in units of log2(e); capped scores carry their scale already
     const float sl2 = CAP ? 1.4426950408889634f : scale * 1.4426950408889634f;
     const float cap_in = CAP ? scale / softcap : 0.0f;
-    constexpr int OC = HD / 2;                 // output columns of this thread
+    constexpr int OC = HV / 2;                 // output columns of this thread
     float acc[OC];
 #pragma unroll
     for (int c = 0; c < OC; ++c) acc[c] = 0.0f;
@@ -375,7 +382,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
 #pragma unroll
       for (int c = 0; c < OC / 32; ++c) {
         uint32_t ov[32];
-        tc05_ld_32x32b_x32(lane_addr + L::O_COL + b * HD + half * OC + c * 32, ov);
+        tc05_ld_32x32b_x32(lane_addr + L::O_COL + b * HV + half * OC + c * 32, ov);
         tc05_wait_ld();
 #pragma unroll
         for (int e = 0; e < 32; ++e) acc[c * 32 + e] = fmaf(acc[c * 32 + e], resc, __uint_as_float(ov[e]));
@@ -475,7 +482,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
           unsigned char* vpage = gen + L::Q_BYTES + (j % L::STAGES) * L::STAGE_BYTES + L::K_BYTES +
                                  ((p_end - 1) - (p_begin + 2 * j)) * L::PAGE_BOX;
           const int sm_tid = (warp - 2) * 32 + lane;
-          for (int i = sm_tid; i < (PAGE_TOKENS - tail_row) * 8 * HB; i += 256) {
+          for (int i = sm_tid; i < (PAGE_TOKENS - tail_row) * 8 * VB; i += 256) {
             const int box = i / ((PAGE_TOKENS - tail_row) * 8), rem = i % ((PAGE_TOKENS - tail_row) * 8);
             *reinterpret_cast<uint4*>(vpage + box * (2 * L::PAGE_BOX) + (tail_row + rem / 8) * 128 +
                                       (rem % 8) * 16) = make_uint4(0u, 0u, 0u, 0u);
@@ -500,7 +507,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
     if (n_splits > 1) {
       // partial result of this run of pages: per row the maximum and the sum, then the
       // unnormalised outputs; all in units of this CTA's own maximum
-      constexpr int REC = 2 * TILE_Q + TILE_Q * HD;          // floats per (tile, split)
+      constexpr int REC = 2 * TILE_Q + TILE_Q * HV;          // floats per (tile, split)
       const size_t tile_id = ((size_t)s * gridDim.y + h) * (gridDim.x / max_splits) + tile;
       float* mine = part + (tile_id * max_splits + split) * REC;
       if (ok) {
@@ -508,7 +515,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
           mine[r] = m_run;
           mine[TILE_Q + r] = l_run;
         }
-        float* po = mine + 2 * TILE_Q + (size_t)r * HD + half * OC;
+        float* po = mine + 2 * TILE_Q + (size_t)r * HV + half * OC;
 #pragma unroll
         for (int c = 0; c < OC / 4; ++c)
           *reinterpret_cast<float4*>(po + c * 4) =
@@ -539,7 +546,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
           const float m_i = __ldcg(rec + r);
           const float w = (m_i == -INFINITY) ? 0.0f : nb_exp2(m_i - m_ref);
           l_run = fmaf(__ldcg(rec + TILE_Q + r), w, l_run);
-          const float* po = rec + 2 * TILE_Q + (size_t)r * HD + half * OC;
+          const float* po = rec + 2 * TILE_Q + (size_t)r * HV + half * OC;
 #pragma unroll
           for (int c = 0; c < OC / 4; ++c) {
             const float4 f = __ldcg(reinterpret_cast<const float4*>(po + c * 4));
@@ -563,10 +570,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
         l_run = fmaf(l_run, fix, nb_exp2(sk - m_f));
       }
       const float inv = (l_run > 0.0f ? fix / l_run : 0.0f) * opt.gate_of(row0 + q0 + r, h);
-      TOut* dst = out + (size_t)(row0 + q0 + r) * out_stride + (size_t)h * HD + half * OC;
+      TOut* dst = out + (size_t)(row0 + q0 + r) * out_stride + (size_t)h * dv + half * OC;
       if constexpr (sizeof(TOut) == 2) {
 #pragma unroll
         for (int c = 0; c < OC / 8; ++c) {
+          if (VAR && half * OC + c * 8 >= dv) break;
           uint4 u;
           __nv_bfloat162* hh = reinterpret_cast<__nv_bfloat162*>(&u);
 #pragma unroll
@@ -576,10 +584,12 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
         }
       } else {
 #pragma unroll
-        for (int c = 0; c < OC / 4; ++c)
+        for (int c = 0; c < OC / 4; ++c) {
+          if (VAR && half * OC + c * 4 >= dv) break;
           *reinterpret_cast<float4*>(dst + c * 4) =
               make_float4(acc[c * 4] * inv, acc[c * 4 + 1] * inv, acc[c * 4 + 2] * inv,
                           acc[c * 4 + 3] * inv);
+        }
       }
     }
   }
@@ -610,25 +620,25 @@ int* error_word() {
   return w ? w + NB_ERRW_ATTENTION_PREFILL_TC : nullptr;
 }
 
-template <int HD, typename TOut, bool CAP>
+template <int HK, int HV, typename TOut, bool CAP, bool VAR>
 int launch_tc(const void* q, int q_stride, int q_col, int n_rows, const int* cu_rows,
               const int* seq_slot, const int* seq_pos0, const void* k_cache, const void* v_cache,
               long long n_pages, const int* block_table, int max_pages, int n_heads, int n_kv_heads,
               void* out, int out_stride, float scale, float softcap, const float* sink, NbAttnOpts opt,
               int n_seqs, int max_q_len, int max_splits, int chunk_pages, float* part,
-              int* counters, int append, int k_col, int v_col, cudaStream_t stream) {
-  using L = AttnSmem<HD>;
+              int* counters, int append, int k_col, int v_col, int dk, int dv, cudaStream_t stream) {
+  using L = AttnSmem<HK, HV>;
   CUtensorMap mq, mk, mv, mn;
   int rc = make_map(&mq, q, n_rows, q_stride, TILE_Q, 64, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2);
   if (rc) return rc;
   const long long kv_rows = n_pages * n_kv_heads * PAGE_TOKENS;
-  rc = make_map(&mk, k_cache, kv_rows, HD, PAGE_TOKENS, 64, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2);
+  rc = make_map(&mk, k_cache, kv_rows, dk, PAGE_TOKENS, 64, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2);
   if (rc) return rc;
-  rc = make_map(&mv, v_cache, kv_rows, HD, PAGE_TOKENS, 64, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2);
+  rc = make_map(&mv, v_cache, kv_rows, dv, PAGE_TOKENS, 64, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2);
   if (rc) return rc;
   rc = make_map(&mn, q, n_rows, q_stride, PAGE_TOKENS, 64, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2);
   if (rc) return rc;
-  auto kern = attention_prefill_tc_kernel<HD, TOut, CAP>;
+  auto kern = attention_prefill_tc_kernel<HK, HV, TOut, CAP, VAR>;
   static bool configured = false;   // per instantiation
   if (!configured) {
     NB_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL));
@@ -638,7 +648,7 @@ int launch_tc(const void* q, int q_stride, int q_col, int n_rows, const int* cu_
   NB_CUDA(nb_launch(kern, grid, dim3(TC_THREADS), (size_t)L::TOTAL, stream, mq, mk, mv, mn, append, k_col,
                     v_col, q_col, cu_rows, seq_slot, seq_pos0, block_table, max_pages, n_kv_heads,
                     n_heads / n_kv_heads, (TOut*)out, out_stride, scale, softcap, sink, opt,
-                    max_splits, chunk_pages, part, counters, error_word()));
+                    max_splits, chunk_pages, part, counters, error_word(), dk, dv));
   return 0;
 }
 
@@ -653,6 +663,15 @@ NB_EXPORT int nb_attention_prefill_tc_supported(int dtype, int head_dim, int n_h
   if (q_stride % 8 != 0 || q_col % 8 != 0) return 0;            // TMA: 16-byte pitch and start
   if (out_stride % (out_dtype == NB_F32 ? 4 : 8) != 0) return 0;  // 16-byte output stores
   return head_dim == 64 || head_dim == 128;
+}
+
+// 1 if its variant for keys of d and values of dv numbers takes this shape.
+NB_EXPORT int nb_attention_prefill_tc_mixed_supported(int dtype, int d, int dv, int n_heads,
+                                                      int n_kv_heads, int page, int q_stride,
+                                                      int q_col, int out_dtype, int out_stride) {
+  if (d % 8 != 0 || dv % 8 != 0 || d < 8 || dv < 8 || d > 128 || dv > 128 || out_dtype != NB_BF16) return 0;
+  return nb_attention_prefill_tc_supported(dtype, 64, n_heads, n_kv_heads, page, q_stride, q_col,
+                                           out_dtype, out_stride);
 }
 
 // Waits for the device, then reads (and lowers) the word that a timed-out wait of this kernel
@@ -673,7 +692,7 @@ NB_EXPORT int nb_attention_prefill_tc_set_wait_budget(long long cycles) {
 }
 
 // Floats of scratch per (sequence, head, 128-row tile, split) when the pages of a tile are cut
-// into more than one run.
+// into more than one run (head_dim: of the values, 64 or 128 as staged).
 NB_EXPORT int nb_attention_prefill_tc_record(int head_dim) { return 2 * TILE_Q + TILE_Q * head_dim; }
 
 // Rows of sequence s are cu_rows[s]..cu_rows[s+1] of the packed batch (n_rows rows of q_stride
@@ -686,6 +705,7 @@ NB_EXPORT int nb_attention_prefill_tc_record(int head_dim) { return 2 * TILE_Q +
 // head after head); every seq_pos0 must then be a multiple of the page size, and the kernel
 // writes them to the cache itself.  softcap > 0: a score becomes softcap * tanh(score /
 // softcap); sink: fp32 [n_heads] logits of one more term of the softmax's denominator, or null.
+// value_dim: the size of a value where it is not the key's head_dim (no append, no cap then).
 // window / keep_first / mask_block, gate: the options of NbAttnOpts.  With kept first tokens (window > 0 and
 // keep_first > 0) the last of the max_splits runs is theirs: max_splits >= 2, and the runs before
 // it, max_splits - 1 of chunk_pages pages, must cover what a tile's window spans.
@@ -693,7 +713,7 @@ NB_EXPORT int nb_attention_prefill_tc_masked(const void* q, int dtype, int q_str
                                       const int* cu_rows, const int* seq_slot, const int* seq_pos0,
                                       const void* k_cache, const void* v_cache, int n_pages,
                                       const int* block_table, int max_pages, int page, int n_heads,
-                                      int n_kv_heads, int head_dim, void* out, int out_dtype,
+                                      int n_kv_heads, int head_dim, int value_dim, void* out, int out_dtype,
                                       int out_stride, float scale, float softcap,
                                       const float* sink, int window, int keep_first, int mask_block,
                                       const float* gate, int gate_stride, int gate_col,
@@ -706,11 +726,15 @@ NB_EXPORT int nb_attention_prefill_tc_masked(const void* q, int dtype, int q_str
   const NbAttnOpts opt{window, keep_first, mask_block, gate, gate_stride, gate_col};
   NB_REQUIRE(!opt.keeps() || max_splits >= 2, NB_ERR_BAD_ARG,
              "attention_prefill_tc: kept first tokens take a run of their own");
-  NB_REQUIRE(nb_attention_prefill_tc_supported(dtype, head_dim, n_heads, n_kv_heads, page, q_stride,
-                                               q_col, out_dtype, out_stride),
+  const bool mixed = value_dim != head_dim;
+  NB_REQUIRE(mixed ? nb_attention_prefill_tc_mixed_supported(dtype, head_dim, value_dim, n_heads, n_kv_heads,
+                                                             page, q_stride, q_col, out_dtype, out_stride) &&
+                         !append && softcap == 0.0f
+                   : nb_attention_prefill_tc_supported(dtype, head_dim, n_heads, n_kv_heads, page, q_stride,
+                                                       q_col, out_dtype, out_stride),
              NB_ERR_UNSUPPORTED,
-             "attention_prefill_tc: unsupported shape (head size %d, %d/%d heads, row pitch %d)",
-             head_dim, n_heads, n_kv_heads, q_stride);
+             "attention_prefill_tc: unsupported shape (head sizes %d/%d, %d/%d heads, row pitch %d)",
+             head_dim, value_dim, n_heads, n_kv_heads, q_stride);
   NB_REQUIRE(n_seqs <= 65535 && n_heads <= 65535 && n_rows > 0 && n_pages > 0, NB_ERR_UNSUPPORTED,
              "attention_prefill_tc: bad sizes");
   NB_REQUIRE(!append || (k_col % 8 == 0 && v_col % 8 == 0 && k_col >= 0 && v_col >= 0),
@@ -728,17 +752,24 @@ NB_EXPORT int nb_attention_prefill_tc_masked(const void* q, int dtype, int q_str
                  (uintptr_t)out % 16 == 0,
              NB_ERR_UNSUPPORTED, "attention_prefill_tc: operands must be 16-byte aligned");
   int rc = NB_ERR_UNSUPPORTED;
-#define NB_ARGS q, q_stride, q_col, n_rows, cu_rows, seq_slot, seq_pos0, k_cache, v_cache, (long long)n_pages, block_table, max_pages, n_heads, n_kv_heads, out, out_stride, scale, softcap, sink, opt, n_seqs, max_q_len, max_splits, chunk_pages, part, counters, append, k_col, v_col, stream
+#define NB_ARGS q, q_stride, q_col, n_rows, cu_rows, seq_slot, seq_pos0, k_cache, v_cache, (long long)n_pages, block_table, max_pages, n_heads, n_kv_heads, out, out_stride, scale, softcap, sink, opt, n_seqs, max_q_len, max_splits, chunk_pages, part, counters, append, k_col, v_col, head_dim, value_dim, stream
   NB_REQUIRE(softcap >= 0.0f, NB_ERR_BAD_ARG, "attention_prefill_tc: a cap is positive, or 0 for none");
-  if (softcap > 0.0f) {
-    if (head_dim == 64)
-      rc = out_dtype == NB_F32 ? launch_tc<64, float, true>(NB_ARGS) : launch_tc<64, bf16, true>(NB_ARGS);
-    else
-      rc = out_dtype == NB_F32 ? launch_tc<128, float, true>(NB_ARGS) : launch_tc<128, bf16, true>(NB_ARGS);
-  } else if (head_dim == 64)
-    rc = out_dtype == NB_F32 ? launch_tc<64, float, false>(NB_ARGS) : launch_tc<64, bf16, false>(NB_ARGS);
-  else
-    rc = out_dtype == NB_F32 ? launch_tc<128, float, false>(NB_ARGS) : launch_tc<128, bf16, false>(NB_ARGS);
+#define NB_ONE(HD_, CAP_)                                                                      \
+  rc = out_dtype == NB_F32 ? launch_tc<HD_, HD_, float, CAP_, false>(NB_ARGS)                  \
+                           : launch_tc<HD_, HD_, bf16, CAP_, false>(NB_ARGS)
+  if (mixed) {
+    if (head_dim <= 64 && value_dim <= 64) rc = launch_tc<64, 64, bf16, false, true>(NB_ARGS);
+    else if (head_dim <= 64) rc = launch_tc<64, 128, bf16, false, true>(NB_ARGS);
+    else if (value_dim <= 64) rc = launch_tc<128, 64, bf16, false, true>(NB_ARGS);
+    else rc = launch_tc<128, 128, bf16, false, true>(NB_ARGS);
+  } else if (softcap > 0.0f) {
+    if (head_dim == 64) NB_ONE(64, true);
+    else NB_ONE(128, true);
+  } else {
+    if (head_dim == 64) NB_ONE(64, false);
+    else NB_ONE(128, false);
+  }
+#undef NB_ONE
 #undef NB_ARGS
   if (rc) return rc;
   NB_CHECK_LAUNCH("attention_prefill_tc");
@@ -758,7 +789,7 @@ NB_EXPORT int nb_attention_prefill_tc_capped(const void* q, int dtype, int q_str
                                       cudaStream_t stream) {
   return nb_attention_prefill_tc_masked(q, dtype, q_stride, q_col, n_rows, cu_rows, seq_slot, seq_pos0,
                                         k_cache, v_cache, n_pages, block_table, max_pages, page,
-                                        n_heads, n_kv_heads, head_dim, out, out_dtype, out_stride,
+                                        n_heads, n_kv_heads, head_dim, head_dim, out, out_dtype, out_stride,
                                         scale, softcap, sink, window, 0, 0, nullptr, 0, 0, n_seqs,
                                         max_q_len, max_splits, chunk_pages, part, counters, append,
                                         k_col, v_col, stream);

@@ -275,4 +275,5 @@ struct NbPagedKV {
   int page;                 // tokens per page
   int n_kv_heads;
   int head_dim;
+  int value_dim;            // of the V plane, where a kernel takes one of another size (else unused)
 };

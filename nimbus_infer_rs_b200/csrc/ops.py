@@ -865,13 +865,36 @@ class CudaBackend:
                        int(chunk), _ptr(gate), gate.shape[1] if gate is not None else 0, int(gate_col),
                        n, n_splits, _ptr(acc), _ptr(ml), _ptr(counters), self._stream())
             return
-        if one_size and q.dtype == k_store.k.dtype and not layout.is_decode and self.use_tcgen05 \
-                and scale > 0 and self.lib.nb_attention_prefill_tc_supported(
+        if shared and not one_size and q.dtype == k_store.k.dtype and layout.is_decode and \
+                out.dtype == torch.bfloat16 and q.shape[1] % 8 == 0 and \
+                self.lib.nb_attention_decode_mixed_supported(code, d, dv, n_heads, k_store.n_kv_heads,
+                                                             k_store.page):
+            # the same for keys and values of different sizes in one store
+            pages = max(1, -(-layout.max_kv_len // k_store.page))
+            if look_back > 0:
+                pages = min(pages, (look_back + k_store.page - 1) // k_store.page + 1)
+            row = self.lib.nb_attention_decode_mixed_row(d, dv)
+            n_splits = decode_splits(n * k_store.n_kv_heads, pages, k_store.page, row, self._sms,
+                                     self._cluster_limit if self.decode_clusters else 16) + (1 if keeps else 0)
+            acc, ml, counters = self._decode_scratch(q.device, n, n_heads, k_store.n_kv_heads, row, n_splits)
+            self._call("nb_attention_decode_mixed", _ptr(q), q.shape[1], _ptr(layout.row_slot),
+                       _ptr(layout.row_pos), _ptr(k_store.k), _ptr(k_store.v), _ptr(k_store.block_table),
+                       k_store.block_table.shape[1], k_store.page, n_heads, k_store.n_kv_heads, d, dv,
+                       _ptr(out), out.shape[1], float(scale), float(softcap or 0.0), _ptr(sink),
+                       int(window), int(keep_first), int(chunk), _ptr(gate),
+                       gate.shape[1] if gate is not None else 0, int(gate_col), n, n_splits, _ptr(acc),
+                       _ptr(ml), _ptr(counters), self.decode_clusters, self._stream())
+            return
+        if shared and q.dtype == k_store.k.dtype and not layout.is_decode and self.use_tcgen05 and scale > 0 and (
+                self.lib.nb_attention_prefill_tc_supported(
                     code, d, n_heads, k_store.n_kv_heads, k_store.page, q.shape[1], 0,
-                    dtype_code(out.dtype), out.shape[1]):
-            # prompts in bfloat16 with heads of 64 or 128: tcgen05 tiles of 128 rows; the pages a
-            # tile reads are cut into runs when CTAs would idle, and kept first tokens that lie
-            # before a tile's window are one more run
+                    dtype_code(out.dtype), out.shape[1]) if one_size else
+                not softcap and self.lib.nb_attention_prefill_tc_mixed_supported(
+                    code, d, dv, n_heads, k_store.n_kv_heads, k_store.page, q.shape[1], 0,
+                    dtype_code(out.dtype), out.shape[1])):
+            # prompts in bfloat16 with heads of 64 or 128, or keys and values of different sizes:
+            # tcgen05 tiles of 128 rows; the pages a tile reads are cut into runs when CTAs would
+            # idle, and kept first tokens that lie before a tile's window are one more run
             if layout.n_rows > layout.n_tokens:
                 out[layout.n_tokens:layout.n_rows].zero_()      # padding rows
             tiles = -(-layout.max_q_len // 128)
@@ -886,11 +909,12 @@ class CudaBackend:
             max_splits = runs + (1 if keeps else 0)
             part = counters = None
             if max_splits > 1:
-                part, counters = self._prefill_scratch(q.device, ctas, max_splits, d)
+                staged = d if one_size else (64 if dv <= 64 else 128)
+                part, counters = self._prefill_scratch(q.device, ctas, max_splits, staged)
             self._call("nb_attention_prefill_tc_masked", _ptr(q), code, q.shape[1], 0, q.shape[0],
                        _ptr(layout.cu_rows), _ptr(layout.seq_slot), _ptr(layout.seq_pos0),
                        _ptr(k_store.k), _ptr(k_store.v), k_store.k.shape[0], _ptr(k_store.block_table),
-                       k_store.block_table.shape[1], k_store.page, n_heads, k_store.n_kv_heads, d,
+                       k_store.block_table.shape[1], k_store.page, n_heads, k_store.n_kv_heads, d, dv,
                        _ptr(out), dtype_code(out.dtype), out.shape[1], float(scale),
                        float(softcap or 0.0), _ptr(sink), int(window), int(keep_first), int(chunk),
                        _ptr(gate), gate.shape[1] if gate is not None else 0, int(gate_col),

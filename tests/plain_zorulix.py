@@ -160,12 +160,10 @@ def delta_walk(q, k, v, g, beta, S=None):
     S = q.new_zeros(H, d, dv) if S is None else S.clone()
     out = q.new_zeros(T, H, dv)
     for t in range(T):
-        for h in range(H):
-            s = g[t, h][:, None] * S[h]
-            u = beta[t, h] * (v[t, h] - s.T @ k[t, h])
-            s = s + torch.outer(k[t, h], u)
-            S[h] = s
-            out[t, h] = s.T @ q[t, h]
+        S = g[t][:, :, None] * S
+        u = beta[t][:, None] * (v[t] - torch.einsum("hkv,hk->hv", S, k[t]))
+        S = S + k[t][:, :, None] * u[:, None, :]
+        out[t] = torch.einsum("hkv,hk->hv", S, q[t])
     return out, S
 
 
@@ -214,9 +212,10 @@ def experts_mixed(x, W, p, f, choice=None):
         idx = choice
         w = torch.softmax(torch.gather(z, 1, idx), -1)
     y = torch.zeros_like(x)
-    for t in range(x.shape[0]):
-        for e, s in zip(idx[t].tolist(), w[t]):
-            y[t] = y[t] + s * expert(x[t], W, f"{p}e{e}.")
+    for e in range(z.shape[1]):
+        t, k = (idx == e).nonzero(as_tuple=True)
+        if len(t):
+            y[t] = y[t] + w[t, k][:, None] * expert(x[t], W, f"{p}e{e}.")
     if f.get("shared"):
         y = y + torch.sigmoid(x @ W[p + "shared.sg"].T) * expert(x, W, p + "shared.")
     return y
