@@ -415,11 +415,12 @@ class OpTimer:
         if kind == "scaled_pair_add":
             return nb(a[0], a[2], a[7]) + 2 * nb(a[4]), 0
         if kind == "gated_delta":
-            lay, heads, kv_heads, d, dv, out = a[11], a[13], a[14], a[15], a[16], a[17]
-            # convolved q, k, v, the logits of rate, decay and gate per token, the state of every
+            taps, lay, heads, kv_heads, d, dv, out = a[3], a[15], *a[17:22]
+            # q, k, v, the logits of rate, decay and gate per token, the state of every
             # sequence in and out; per token and head 4 d dv multiply-adds on the CUDA cores
             per_token = 2 * kv_heads * d + heads * (2 * dv + d + 1)
-            return lay.n_tokens * per_token * 4 + nb(out) + 2 * lay.n_seqs * heads * d * dv * 4, \
+            state = heads * d * dv + max(int(taps) - 1, 0) * (2 * kv_heads * d + heads * dv)
+            return lay.n_tokens * per_token * 4 + nb(out) + 2 * lay.n_seqs * state * 4, \
                 2 * 4 * lay.n_tokens * heads * d * dv
         if kind in ("rms_add", "ln_add"):
             return nb(a[0], a[6], a[7]) + 2 * nb(a[3]), 0

@@ -18,16 +18,17 @@
 // so the state is read twice and written once per four tokens, the eight dot products of a column
 // with it are independent of one another, and only the four u_t (a few multiply-adds) follow one
 // another.  Decays are multiplied up, never divided by, so nothing overflows however strong they are.
-//   gated_delta_prepare  a warp per (block of four tokens, head) computes a record: E_3, the four
-//                        (beta_t E_t k_t), (E_t q_t), (k_s E_(s..3)), the numbers A and B, and the
-//                        four beta_t v_t.  A block's missing tokens (a sequence's last block) are
-//                        tokens with k = q = v = 0, g = 1.
+//   gated_delta_prepare  a warp per (block of four tokens, head): the short convolution and silu
+//                        of q, k and v (of projected rows, the inputs before the step from the
+//                        state row), then a record: E_3, the four (beta_t E_t k_t), (E_t q_t),
+//                        (k_s E_(s..3)), the numbers A and B, and the four beta_t v_t.  A block's
+//                        missing tokens (a sequence's last block) are tokens with k = q = v = 0, g = 1.
 //   gated_delta_walk     a CTA takes COLS columns of one (sequence, head); the columns are
-//                        independent.  A group of LPG lanes holds four columns, CH key channels a
-//                        lane, so a number of the record that was read from shared memory meets
-//                        four columns.  The 32 partial sums of a block (four tokens, four columns,
-//                        two products) are reduced over the lanes by halving: each lane ends with
-//                        32 / LPG of them.  Records come through two buffers of asynchronous copies.
+//                        independent.  A group of LPG lanes holds NC columns, CH key channels a
+//                        lane, two neighbouring channels in a register pair (packed multiply-adds).
+//                        The 8 NC partial sums of a block (four tokens, NC columns, two products)
+//                        are reduced over the lanes by halving: each lane ends with 8 NC / LPG of
+//                        them.  Records come through two buffers of asynchronous copies.
 //   delta_finish         norm, weight and gate (the norm needs all of a head's columns).
 // A sequence may be cut into steps anywhere: where blocks begin only changes the rounding.
 //
@@ -44,33 +45,40 @@ constexpr int MAX_DIM = 256;
 
 __device__ __forceinline__ float gd_softplus(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
 
-// Sums of N values over L lanes by halving: afterwards the lane with number q in its group of L
-// holds the sums with indices q * (N / L) .. in v[0 ..] (N >= L), or, when N < L, index q / (L / N).
-template <int N, int L>
-__device__ __forceinline__ void reduce_by_halving(float (&v)[N], int lane) {
+// Sums of N values over L lanes by halving; the lanes are STEP apart and q is the lane's number among
+// them.  Afterwards it holds the sums with indices q * (N / L) .. in v[0 ..] (N >= L), or, when N < L,
+// index q / (L / N).
+template <int N, int L, int STEP>
+__device__ __forceinline__ void reduce_by_halving(float (&v)[N], int q) {
   int n = N;
 #pragma unroll
   for (int m = L / 2; m >= 1; m >>= 1) {
     if (n > 1) {
       n >>= 1;
-      const bool up = (lane & m) != 0;
+      const bool up = (q & m) != 0;
 #pragma unroll
       for (int i = 0; i < N / 2; ++i) {
         if (i < n) {
           const float send = up ? v[i] : v[i + n];
           const float keep = up ? v[i + n] : v[i];
-          v[i] = keep + __shfl_xor_sync(0xffffffffu, send, m);
+          v[i] = keep + __shfl_xor_sync(0xffffffffu, send, m * STEP);
         }
       }
     } else {
-      v[0] += __shfl_xor_sync(0xffffffffu, v[0], m);
+      v[0] += __shfl_xor_sync(0xffffffffu, v[0], m * STEP);
     }
   }
 }
 
 struct Source {               // where a row's numbers lie
-  const float* qkv;           // [rows][qkv_stride]: q heads, k heads, v heads (convolved, activated)
-  int qkv_stride;
+  const float* qkv;           // rows of qkv_stride: q heads, k heads, v heads from column qkv_col
+  int qkv_stride, qkv_col;
+  // taps > 0: those are projections, to be convolved (conv: [channels][taps]; inputs: a slot's last
+  // taps - 1 rows of channels at inputs + slot * in_stride) and activated; 0: they are ready
+  const float* conv;
+  int taps;
+  float* inputs;
+  int in_stride, channels;
   const float* beta;          // [rows][beta_stride], head h's logit at column beta_col + h
   int beta_stride, beta_col;
   const float* low;           // [rows][low_stride]: decay logits at decay_col, gate logits at gate_col
@@ -83,50 +91,123 @@ struct Source {               // where a row's numbers lie
 __host__ __device__ constexpr int record_head(int DP) { return 13 * DP + 32; }
 __host__ __device__ inline int record_floats(int DP, int dvp) { return record_head(DP) + BLK * dvp; }
 
+constexpr int MAX_FUSED_TAPS = 4;
+
+// Four neighbouring channels c .. c+3 (those below `end`) of BLK tokens: y[t] = the ready numbers or
+// silu of the convolution.  base: the channels' first column in a row; ch0: their first channel.
+// CONV: 0 ready, 1 convolved, 2 convolved with the hardware's exponential and reciprocal in the silu
+// (a bfloat16 run, where projections and their activations are rounded anyway).
+template <int CONV>
+__device__ __forceinline__ void take_channels(const Source& src, const float* in_row, int row0, int row1,
+                                              int first, int ch0, int c, int end, bool vec,
+                                              float (&y)[BLK][4]) {
+  auto load4 = [&](const float* p, float (&v)[4]) {
+    if (vec && c < end) {
+      const float4 f = *reinterpret_cast<const float4*>(p);
+      v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+    } else {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v[e] = c + e < end ? p[e] : 0.0f;
+    }
+  };
+  const float* col = src.qkv + src.qkv_col + ch0 + c;
+  if constexpr (CONV == 0) {
+#pragma unroll
+    for (int t = 0; t < BLK; ++t)
+      load4(col + (size_t)(first + t < row1 ? first + t : row0) * src.qkv_stride, y[t]);
+  } else {
+    // inputs first - 3 .. first + 3; weights with zeros in front up to four taps
+    float x[BLK + MAX_FUSED_TAPS - 1][4], w[MAX_FUSED_TAPS][4];
+    const int taps = src.taps;
+#pragma unroll
+    for (int i = 0; i < BLK + MAX_FUSED_TAPS - 1; ++i) {
+      const int r = first - (MAX_FUSED_TAPS - 1) + i;
+      const int back = row0 - r;                 // rows before the step's first: 1 is the newest
+      if (back <= 0) load4(col + (size_t)(r < row1 ? r : row0) * src.qkv_stride, x[i]);
+      else if (back < taps) load4(in_row + (size_t)(taps - 1 - back) * src.channels + ch0 + c, x[i]);
+      else x[i][0] = x[i][1] = x[i][2] = x[i][3] = 0.0f;
+    }
+    if (taps == MAX_FUSED_TAPS && vec && c < end) {          // (the weights of a channel: 16 bytes)
+      const float4* wp = reinterpret_cast<const float4*>(src.conv) + ch0 + c;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float4 f = wp[e];
+        w[0][e] = f.x; w[1][e] = f.y; w[2][e] = f.z; w[3][e] = f.w;
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < MAX_FUSED_TAPS; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int tap = j - (MAX_FUSED_TAPS - taps);
+          w[j][e] = (tap >= 0 && c + e < end) ? src.conv[(size_t)(ch0 + c + e) * taps + tap] : 0.0f;
+        }
+    }
+#pragma unroll
+    for (int t = 0; t < BLK; ++t)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        float v = 0.0f;
+#pragma unroll
+        for (int j = 0; j < MAX_FUSED_TAPS; ++j) v = fmaf(w[j][e], x[t + j][e], v);
+        y[t][e] = CONV == 2 ? nb_silu_fast(v) : nb_silu(v);
+      }
+  }
+}
+
 // A sequence's blocks start at record cu_rows[seq] / 4 + seq, so that no two sequences overlap.
-template <int DP>
+template <int DP, int CONV>
 __global__ void __launch_bounds__(128)
 gated_delta_prepare_kernel(Source src, float key_eps, const int* cu_rows, const int* seq_slot,
-                           float* records, int n_heads, int n_kv_heads, int d, int dv, int vec) {
+                           float* records, int n_heads, int n_kv_heads, int d, int dv, int vec,
+                           int vec_in, int vec_v) {
   nb_grid_dependency_wait();
   nb_launch_dependents();
   constexpr int KIT = (DP + 127) / 128;             // quads of channels a lane holds
   const int seq = blockIdx.z, h = blockIdx.y, lane = threadIdx.x & 31;
   const int blk = blockIdx.x * 4 + (threadIdx.x >> 5);
   const int row0 = cu_rows[seq], row1 = cu_rows[seq + 1];
-  const int first = row0 + blk * BLK;
-  if (seq_slot[seq] < 0 || first >= row1) return;
+  const int first = row0 + blk * BLK, slot = seq_slot[seq];
+  if (slot < 0 || first >= row1) return;
   const int g = h / (n_heads / n_kv_heads);
   const int dvp = (dv + 3) & ~3;
   float* rec = records + ((size_t)(row0 / BLK + seq + blk) * n_heads + h) * record_floats(DP, dvp);
+  const float* in_row = CONV ? src.inputs + (size_t)slot * src.in_stride : nullptr;
   const float rate = expf(src.a_log[h]);
   const float q_scale = 1.0f / sqrtf((float)d);
+  // 16-byte loads of the rows; near the step's start also of the state row
+  const bool vec_q = vec_in && (!CONV || vec || blk > 0);
 
   float k[BLK][KIT * 4], q[BLK][KIT * 4], w[BLK][KIT * 4], beta[BLK];
-  auto load4 = [&](const float* p, int c, float (&v)[KIT * 4], int at) {
-    if (vec && c < d) {
-      const float4 f = *reinterpret_cast<const float4*>(p + c);
-      v[at] = f.x; v[at + 1] = f.y; v[at + 2] = f.z; v[at + 3] = f.w;
-    } else {
 #pragma unroll
-      for (int e = 0; e < 4; ++e) v[at + e] = c + e < d ? p[c + e] : 0.0f;
+  for (int j = 0; j < KIT; ++j) {
+    const int c = (j * 32 + lane) * 4;
+    float y[BLK][4];
+    take_channels<CONV>(src, in_row, row0, row1, first, g * d, c, d, vec_q, y);
+#pragma unroll
+    for (int t = 0; t < BLK; ++t)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) q[t][j * 4 + e] = y[t][e];
+    take_channels<CONV>(src, in_row, row0, row1, first, (n_kv_heads + g) * d, c, d, vec_q, y);
+#pragma unroll
+    for (int t = 0; t < BLK; ++t) {
+      const int r = first + t < row1 ? first + t : row0;
+      const float* dl = src.low + (size_t)r * src.low_stride + src.decay_col + h * d + c;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) k[t][j * 4 + e] = y[t][e];
+      if (vec_in && c < d) {
+        const float4 f = *reinterpret_cast<const float4*>(dl);
+        w[t][j * 4] = f.x; w[t][j * 4 + 1] = f.y; w[t][j * 4 + 2] = f.z; w[t][j * 4 + 3] = f.w;
+      } else {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) w[t][j * 4 + e] = c + e < d ? dl[e] : 0.0f;
+      }
     }
-  };
-#pragma unroll
-  for (int t = 0; t < BLK; ++t) {
-    const int r = first + t;
-    const bool live = r < row1;
-    const float* row = src.qkv + (size_t)(live ? r : row0) * src.qkv_stride;
-    const float* dl = src.low + (size_t)(live ? r : row0) * src.low_stride + src.decay_col + h * d;
-#pragma unroll
-    for (int j = 0; j < KIT; ++j) {
-      const int c = (j * 32 + lane) * 4;
-      load4(row + g * d, c, q[t], j * 4);
-      load4(row + (n_kv_heads + g) * d, c, k[t], j * 4);
-      load4(dl, c, w[t], j * 4);
-    }
-    beta[t] = live ? nb_sigmoid(src.beta[(size_t)r * src.beta_stride + src.beta_col + h]) : 0.0f;
   }
+#pragma unroll
+  for (int t = 0; t < BLK; ++t)
+    beta[t] = first + t < row1
+                  ? nb_sigmoid(src.beta[(size_t)(first + t) * src.beta_stride + src.beta_col + h]) : 0.0f;
   // unit vectors and decays
   float ss[2 * BLK];
 #pragma unroll
@@ -183,7 +264,7 @@ gated_delta_prepare_kernel(Source src, float key_eps, const int* cu_rows, const 
     }
     store(9 + s, kd);
   }
-  reduce_by_halving<16, 32>(ab, lane);           // lane l holds number l / 2
+  reduce_by_halving<16, 32, 1>(ab, lane);           // lane l holds number l / 2
   {
     const int t = (lane & 15) >> 2, s = lane & 3;   // slot `lane`: A (0..15), B (16..31), row t, column s
     const bool is_b = lane >= 16, there = is_b ? s <= t : s < t;
@@ -208,42 +289,91 @@ gated_delta_prepare_kernel(Source src, float key_eps, const int* cu_rows, const 
   store(0, w[BLK - 1]);
   // beta_t v_t
   float* vd = rec + record_head(DP);
+  for (int c = lane * 4; c < dvp; c += 128) {
+    float y[BLK][4];
+    take_channels<CONV>(src, in_row, row0, row1, first, 2 * n_kv_heads * d + h * dv, c, dv,
+                        vec_v && (!CONV || vec || blk > 0), y);
 #pragma unroll
-  for (int t = 0; t < BLK; ++t) {
-    const int r = first + t;
-    const float* v = src.qkv + (size_t)(r < row1 ? r : row0) * src.qkv_stride + 2 * n_kv_heads * d + h * dv;
-    for (int c = lane; c < dvp; c += 32)
-      vd[t * dvp + c] = (r < row1 && c < dv) ? beta[t] * v[c] : 0.0f;
+    for (int t = 0; t < BLK; ++t) {
+      const float b = beta[t];                     // zero for a missing token
+      *reinterpret_cast<float4*>(vd + t * dvp + c) =
+          make_float4(b * y[t][0], b * y[t][1], b * y[t][2], b * y[t][3]);
+    }
   }
 }
 
-// CH: key channels a lane holds for each of its four columns; LPG: lanes of a group; NW: warps.
-template <int CH, int LPG, int NW>
+// two fp32 numbers in a register pair
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pair_of(float lo, float hi) {
+  f32x2 r;
+  asm("mov.b64 %0, {%1, %2};\n" : "=l"(r) : "f"(lo), "f"(hi));
+  return r;
+}
+__device__ __forceinline__ float2 unpair(f32x2 v) {
+  float2 f;
+  asm("mov.b64 {%0, %1}, %2;\n" : "=f"(f.x), "=f"(f.y) : "l"(v));
+  return f;
+}
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+  f32x2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;\n" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+  f32x2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;\n" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+
+// NC numbers that lie side by side
+template <int NC>
+__device__ __forceinline__ void load_cols(const float* p, float (&v)[NC]) {
+  if constexpr (NC == 4) {
+    const float4 f = *reinterpret_cast<const float4*>(p);
+    v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+  } else {
+    const float2 f = *reinterpret_cast<const float2*>(p);
+    v[0] = f.x; v[1] = f.y;
+  }
+}
+template <int NC>
+__device__ __forceinline__ void store_cols(float* p, const float (&v)[NC]) {
+  if constexpr (NC == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  else *reinterpret_cast<float2*>(p) = make_float2(v[0], v[1]);
+}
+
+// CH: key channels a lane holds for each of its NC columns; LPG: lanes of a group; NW: warps.
+template <int CH, int LPG, int NC, int NW>
 struct Walk {
   static constexpr int DP = CH * LPG;
-  static constexpr int GROUPS = NW * (32 / LPG);
-  static constexpr int COLS = 4 * GROUPS;
+  static constexpr int GPW = 32 / LPG;                           // groups of a warp
+  static constexpr int GROUPS = NW * GPW;
+  static constexpr int COLS = NC * GROUPS;
+  static constexpr int V = 2 * BLK * NC;                         // sums of a block and group
   static constexpr int SB = DP > 128 ? 2 : 4;                    // blocks a buffer holds
   static constexpr int BUF = SB * (record_head(DP) + BLK * COLS);  // floats of a buffer
-  static constexpr int SMEM = (2 * BUF + 2 * GROUPS * 32) * 4;
+  static constexpr int SMEM = (2 * BUF + 2 * GROUPS * V) * 4;
 };
 
-template <int CH, int LPG, int NW>
+template <int CH, int LPG, int NC, int NW>
 __global__ void __launch_bounds__(NW * 32)
 gated_delta_walk_kernel(const float* records, const int* cu_rows, const int* seq_slot, float* state,
                         int state_stride, float* o_raw, int n_heads, int d, int dv, int vec) {
-  using W = Walk<CH, LPG, NW>;
+  using W = Walk<CH, LPG, NC, NW>;
   constexpr int DP = W::DP, COLS = W::COLS, SB = W::SB, THREADS = NW * 32, HEAD = record_head(DP);
-  static_assert(CH % 4 == 0, "a lane takes its channels four at a time");
+  constexpr int GPW = W::GPW, V = W::V;
+  static_assert(CH % 4 == 0 && COLS % 4 == 0 && LPG >= BLK && V >= LPG && (NC == 2 || NC == 4),
+                "a lane takes its channels four at a time");
   nb_grid_dependency_wait();
   extern __shared__ __align__(16) float sm[];
-  float* red = sm + 2 * W::BUF;                     // [2][groups][32]
+  float* red = sm + 2 * W::BUF;                     // [2][groups][V]
   const int col0 = blockIdx.x * COLS, h = blockIdx.y, seq = blockIdx.z, tid = threadIdx.x;
   const int row0 = cu_rows[seq], row1 = cu_rows[seq + 1];
   const int slot = seq_slot[seq];
   if (slot < 0 || row1 <= row0) return;
-  const int lane = tid & 31, group = tid / LPG, q = tid % LPG;
-  const int col = col0 + group * 4;                 // this group's four columns
+  // the groups of a warp lie in turn over its lanes: neighbours read the same numbers of a record
+  const int lane = tid & 31, group = (tid >> 5) * GPW + lane % GPW, q = lane / GPW;
+  const int col = col0 + group * NC;                // this group's columns
   const int dvp = (dv + 3) & ~3, rec_floats = record_floats(DP, dvp);
   const int n_blocks = (row1 - row0 + BLK - 1) / BLK;
   const float* recs = records + ((size_t)(row0 / BLK + seq) * n_heads + h) * rec_floats;
@@ -256,7 +386,7 @@ gated_delta_walk_kernel(const float* records, const int* cu_rows, const int* seq
     for (int b = 0; b < nb; ++b) {
       const float* rec = recs + (size_t)(b0 + b) * rec_step;
       for (int i = tid; i < HEAD / 4; i += THREADS) cp_async16(dst + b * HEAD + i * 4, rec + i * 4);
-      for (int i = tid; i < BLK * COLS / 4; i += THREADS) {
+      for (int i = tid; i < COLS; i += THREADS) {   // BLK rows of COLS / 4 pieces
         const int t = i / (COLS / 4), c = (i % (COLS / 4)) * 4;
         if (col0 + c < dvp)
           cp_async16(dst + SB * HEAD + (b * BLK + t) * COLS + c, rec + HEAD + t * dvp + col0 + c);
@@ -266,135 +396,159 @@ gated_delta_walk_kernel(const float* records, const int* cu_rows, const int* seq
   };
   fetch(0, 0);
 
-  // key channel of state number i of this lane: groups of four, dealt out to the lanes in turn
-  auto channel = [q](int i) { return (((i >> 2) * LPG + q) << 2) + (i & 3); };
-  float S[CH][4];
+  // key channels of pair number i of this lane: quads of channels, dealt out to the lanes in turn
+  auto channel = [q](int i) { return (((i >> 1) * LPG + q) << 2) + 2 * (i & 1); };
+  f32x2 S[CH / 2][NC];                              // [channel pair][column]
 #pragma unroll
-  for (int i = 0; i < CH; ++i) {
-    const int c = channel(i);
-    S[i][0] = S[i][1] = S[i][2] = S[i][3] = 0.0f;
-    if (c >= d || col >= dv) continue;
-    if (vec) {
-      const float4 f = *reinterpret_cast<const float4*>(st + (size_t)c * dv + col);
-      S[i][0] = f.x; S[i][1] = f.y; S[i][2] = f.z; S[i][3] = f.w;
-    } else {
+  for (int i = 0; i < CH / 2; ++i) {
+    float v[2][NC];
 #pragma unroll
-      for (int j = 0; j < 4; ++j)
-        if (col + j < dv) S[i][j] = st[(size_t)c * dv + col + j];
+    for (int e = 0; e < 2; ++e) {
+      const int c = channel(i) + e;
+#pragma unroll
+      for (int j = 0; j < NC; ++j) v[e][j] = 0.0f;
+      if (c < d && col < dv) {
+        if (vec) {
+          load_cols<NC>(st + (size_t)c * dv + col, v[e]);
+        } else {
+#pragma unroll
+          for (int j = 0; j < NC; ++j)
+            if (col + j < dv) v[e][j] = st[(size_t)c * dv + col + j];
+        }
+      }
     }
+#pragma unroll
+    for (int j = 0; j < NC; ++j) S[i][j] = pair_of(v[0][j], v[1][j]);
   }
 
-  int parity = 0;
+  // this lane's output: token q of a block (the first BLK lanes of a group)
+  float* o_at = o_raw + ((size_t)(row0 + q) * n_heads + h) * dv + col;
+  const size_t o_step = (size_t)BLK * n_heads * dv;
+  const int o_rows = q < BLK && col < dv ? row1 - row0 - q : 0;    // tokens there are for it
+  int parity = 0, token = 0;
   for (int b0 = 0, buf = 0; b0 < n_blocks; b0 += SB, buf ^= 1) {
     cp_async_wait<0>();
     __syncthreads();                 // the buffer is in, and every thread has left the other one
     if (b0 + SB < n_blocks) fetch(b0 + SB, buf ^ 1);
     const float* head = sm + buf * W::BUF;
-    const float* vals = head + SB * HEAD + group * 4;
+    const float* vals = head + SB * HEAD + group * NC;
     const int nb = min(SB, n_blocks - b0);
     for (int b = 0; b < nb; ++b, head += HEAD, vals += BLK * COLS) {
-      // r[t][c] = (beta E k)_t . S_c at 4 t + c,  (E q)_t . S_c at 16 + 4 t + c
-      float p[32];
+      // (beta E k)_t . S_c at t NC + c,  (E q)_t . S_c at V / 2 + t NC + c
+      f32x2 acc[V];
 #pragma unroll
-      for (int i = 0; i < 32; ++i) p[i] = 0.0f;
+      for (int i = 0; i < V; ++i) acc[i] = 0ull;
 #pragma unroll
       for (int g = 0; g < CH / 4; ++g) {
 #pragma unroll
         for (int t = 0; t < BLK; ++t) {
-          const float4 kk = *reinterpret_cast<const float4*>(head + (1 + t) * DP + (g * LPG + q) * 4);
-          const float4 qq = *reinterpret_cast<const float4*>(head + (5 + t) * DP + (g * LPG + q) * 4);
+          const ulonglong2 kk = *reinterpret_cast<const ulonglong2*>(head + (1 + t) * DP + (g * LPG + q) * 4);
+          const ulonglong2 qq = *reinterpret_cast<const ulonglong2*>(head + (5 + t) * DP + (g * LPG + q) * 4);
 #pragma unroll
-          for (int c = 0; c < 4; ++c) {
-            p[4 * t + c] = fmaf(kk.x, S[4 * g][c], p[4 * t + c]);
-            p[4 * t + c] = fmaf(kk.y, S[4 * g + 1][c], p[4 * t + c]);
-            p[4 * t + c] = fmaf(kk.z, S[4 * g + 2][c], p[4 * t + c]);
-            p[4 * t + c] = fmaf(kk.w, S[4 * g + 3][c], p[4 * t + c]);
-            p[16 + 4 * t + c] = fmaf(qq.x, S[4 * g][c], p[16 + 4 * t + c]);
-            p[16 + 4 * t + c] = fmaf(qq.y, S[4 * g + 1][c], p[16 + 4 * t + c]);
-            p[16 + 4 * t + c] = fmaf(qq.z, S[4 * g + 2][c], p[16 + 4 * t + c]);
-            p[16 + 4 * t + c] = fmaf(qq.w, S[4 * g + 3][c], p[16 + 4 * t + c]);
+          for (int c = 0; c < NC; ++c) {
+            f32x2& r = acc[t * NC + c];
+            f32x2& o = acc[V / 2 + t * NC + c];
+            r = fma2(kk.x, S[2 * g][c], r);
+            r = fma2(kk.y, S[2 * g + 1][c], r);
+            o = fma2(qq.x, S[2 * g][c], o);
+            o = fma2(qq.y, S[2 * g + 1][c], o);
           }
         }
       }
-      reduce_by_halving<32, LPG>(p, lane);
-      float* mine = red + (parity * W::GROUPS + group) * 32;
+      float p[V];
+#pragma unroll
+      for (int i = 0; i < V; ++i) {
+        const float2 f = unpair(acc[i]);
+        p[i] = f.x + f.y;
+      }
+      reduce_by_halving<V, LPG, GPW>(p, q);
+      float* mine = red + (parity * W::GROUPS + group) * V;
       parity ^= 1;
 #pragma unroll
-      for (int i = 0; i < 32 / LPG; ++i) mine[q * (32 / LPG) + i] = p[i];
+      for (int i = 0; i < V / LPG; ++i) mine[q * (V / LPG) + i] = p[i];
       __syncwarp();
-      // the four u, then the state
-      float u[BLK][4];
+      // the four u
+      float u[BLK][NC];
 #pragma unroll
       for (int t = 0; t < BLK; ++t) {
-        const float4 rr = *reinterpret_cast<const float4*>(mine + 4 * t);
-        const float4 vv = *reinterpret_cast<const float4*>(vals + t * COLS);
-        u[t][0] = vv.x - rr.x; u[t][1] = vv.y - rr.y; u[t][2] = vv.z - rr.z; u[t][3] = vv.w - rr.w;
-        if (t == 0) continue;
-        const float4 a = *reinterpret_cast<const float4*>(head + 13 * DP + 4 * t);
-        const float at[3] = {a.x, a.y, a.z};
+        float r[NC];
+        load_cols<NC>(mine + t * NC, r);
+        load_cols<NC>(vals + t * COLS, u[t]);
+        float4 a = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (t > 0) a = *reinterpret_cast<const float4*>(head + 13 * DP + 4 * t);
 #pragma unroll
-        for (int s = 0; s < t; ++s)
-#pragma unroll
-          for (int c = 0; c < 4; ++c) u[t][c] = fmaf(-at[s], u[s][c], u[t][c]);
+        for (int c = 0; c < NC; ++c) {
+          u[t][c] -= r[c];
+          if (t > 0) u[t][c] = fmaf(-a.x, u[0][c], u[t][c]);
+          if (t > 1) u[t][c] = fmaf(-a.y, u[1][c], u[t][c]);
+          if (t > 2) u[t][c] = fmaf(-a.z, u[2][c], u[t][c]);
+        }
       }
+      // the state
+      f32x2 uu[BLK][NC];
+#pragma unroll
+      for (int t = 0; t < BLK; ++t)
+#pragma unroll
+        for (int c = 0; c < NC; ++c) uu[t][c] = pair_of(u[t][c], u[t][c]);
 #pragma unroll
       for (int g = 0; g < CH / 4; ++g) {
-        const float4 w = *reinterpret_cast<const float4*>(head + (g * LPG + q) * 4);
+        const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(head + (g * LPG + q) * 4);
 #pragma unroll
-        for (int c = 0; c < 4; ++c) {
-          S[4 * g][c] *= w.x;
-          S[4 * g + 1][c] *= w.y;
-          S[4 * g + 2][c] *= w.z;
-          S[4 * g + 3][c] *= w.w;
+        for (int c = 0; c < NC; ++c) {
+          S[2 * g][c] = mul2(w.x, S[2 * g][c]);
+          S[2 * g + 1][c] = mul2(w.y, S[2 * g + 1][c]);
         }
 #pragma unroll
-        for (int s = 0; s < BLK; ++s) {
-          const float4 kk = *reinterpret_cast<const float4*>(head + (9 + s) * DP + (g * LPG + q) * 4);
+        for (int t = 0; t < BLK; ++t) {
+          const ulonglong2 kk = *reinterpret_cast<const ulonglong2*>(head + (9 + t) * DP + (g * LPG + q) * 4);
 #pragma unroll
-          for (int c = 0; c < 4; ++c) {
-            S[4 * g][c] = fmaf(kk.x, u[s][c], S[4 * g][c]);
-            S[4 * g + 1][c] = fmaf(kk.y, u[s][c], S[4 * g + 1][c]);
-            S[4 * g + 2][c] = fmaf(kk.z, u[s][c], S[4 * g + 2][c]);
-            S[4 * g + 3][c] = fmaf(kk.w, u[s][c], S[4 * g + 3][c]);
+          for (int c = 0; c < NC; ++c) {
+            S[2 * g][c] = fma2(kk.x, uu[t][c], S[2 * g][c]);
+            S[2 * g + 1][c] = fma2(kk.y, uu[t][c], S[2 * g + 1][c]);
           }
         }
       }
-      // a token's four outputs: lane t of the group has token t
-      if (q < BLK) {
-        const float4 oo = *reinterpret_cast<const float4*>(mine + 16 + 4 * q);
+      // a token's outputs: lane t of the group has token t
+      if (token < o_rows) {
+        float o[NC];
+        load_cols<NC>(mine + V / 2 + q * NC, o);
         const float4 bb = *reinterpret_cast<const float4*>(head + 13 * DP + 16 + 4 * q);
-        float o[4] = {oo.x, oo.y, oo.z, oo.w};
-        const float bt[4] = {bb.x, bb.y, bb.z, bb.w};
 #pragma unroll
-        for (int s = 0; s < BLK; ++s)
+        for (int c = 0; c < NC; ++c)
+          o[c] = fmaf(bb.x, u[0][c], fmaf(bb.y, u[1][c], fmaf(bb.z, u[2][c], fmaf(bb.w, u[3][c], o[c]))));
+        if (vec) {
+          store_cols<NC>(o_at, o);
+        } else {
 #pragma unroll
-          for (int c = 0; c < 4; ++c) o[c] = fmaf(bt[s], u[s][c], o[c]);
-        const int r = row0 + (b0 + b) * BLK + q;
-        if (r < row1) {
-          float* dst = o_raw + ((size_t)r * n_heads + h) * dv + col;
-          if (vec && col < dv) {
-            *reinterpret_cast<float4*>(dst) = make_float4(o[0], o[1], o[2], o[3]);
-          } else {
-#pragma unroll
-            for (int c = 0; c < 4; ++c)
-              if (col + c < dv) dst[c] = o[c];
-          }
+          for (int c = 0; c < NC; ++c)
+            if (col + c < dv) o_at[c] = o[c];
         }
       }
+      token += BLK;
+      o_at += o_step;
     }
   }
   nb_launch_dependents();
 #pragma unroll
-  for (int i = 0; i < CH; ++i) {
-    const int c = channel(i);
-    if (c >= d || col >= dv) continue;
-    if (vec) {
-      *reinterpret_cast<float4*>(st + (size_t)c * dv + col) =
-          make_float4(S[i][0], S[i][1], S[i][2], S[i][3]);
-    } else {
+  for (int i = 0; i < CH / 2; ++i) {
+    float v[2][NC];
 #pragma unroll
-      for (int j = 0; j < 4; ++j)
-        if (col + j < dv) st[(size_t)c * dv + col + j] = S[i][j];
+    for (int j = 0; j < NC; ++j) {
+      const float2 f = unpair(S[i][j]);
+      v[0][j] = f.x;
+      v[1][j] = f.y;
+    }
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int c = channel(i) + e;
+      if (c >= d || col >= dv) continue;
+      if (vec) {
+        store_cols<NC>(st + (size_t)c * dv + col, v[e]);
+      } else {
+#pragma unroll
+        for (int j = 0; j < NC; ++j)
+          if (col + j < dv) st[(size_t)c * dv + col + j] = v[e][j];
+      }
     }
   }
 }
@@ -446,7 +600,7 @@ gated_delta_step_kernel(Source src, float key_eps, const float* __restrict__ nor
   // store into another CTA's shared memory
   asm volatile("barrier.cluster.arrive.relaxed.aligned;\n" ::: "memory");
 
-  const float* row = src.qkv + (size_t)r * src.qkv_stride;
+  const float* row = src.qkv + (size_t)r * src.qkv_stride + src.qkv_col;
   float v4[4];
 #pragma unroll
   for (int j = 0; j < 4; ++j) v4[j] = col + j < dv ? row[2 * n_kv_heads * d + h * dv + col + j] : 0.0f;
@@ -562,12 +716,12 @@ gated_delta_step_kernel(Source src, float key_eps, const float* __restrict__ nor
   }
 }
 
-template <int CH, int LPG, int NW>
+template <int CH, int LPG, int NC, int NW>
 int launch_walk(cudaStream_t stream, const float* records, const int* cu_rows, const int* seq_slot,
                 float* state, int state_stride, float* o_raw, int n_heads, int d, int dv, int vec,
                 int n_seqs, bool long_walk) {
-  using W = Walk<CH, LPG, NW>;
-  auto kern = gated_delta_walk_kernel<CH, LPG, NW>;
+  using W = Walk<CH, LPG, NC, NW>;
+  auto kern = gated_delta_walk_kernel<CH, LPG, NC, NW>;
   static bool configured = false;   // per instantiation
   if (!configured && W::SMEM > 48 * 1024) {
     NB_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, W::SMEM));
@@ -605,13 +759,16 @@ NB_EXPORT long long nb_gated_delta_scratch(int n_rows, int n_seqs, int n_heads, 
   return (long long)(n_rows / BLK + n_seqs + 1) * n_heads * record_floats(padded_key(d), (dv + 3) & ~3);
 }
 
-// qkv: fp32 [rows][qkv_stride], q heads (n_kv_heads * d), k heads, v heads (n_heads * dv), convolved
-// and activated; beta: fp32 rows, head h's logit at column beta_col + h; low: fp32 rows with the
-// decay logits (n_heads * d) at decay_col and the gate logits (n_heads * dv) at gate_col; a_log
-// [n_heads], dt_bias [n_heads*d], norm_w [dv]; state: a slot's row at state + slot * state_stride
-// holds [n_heads][d][dv] (key channel, value channel); records: scratch (nb_gated_delta_scratch);
-// o_raw: fp32 scratch [n_rows][n_heads*dv]; out: [n_rows][n_heads*dv].
-NB_EXPORT int nb_gated_delta(const float* qkv, int qkv_stride, const float* beta, int beta_stride,
+// qkv: fp32 rows, q heads (n_kv_heads * d), k heads, v heads (n_heads * dv) from column qkv_col: with
+// taps > 0 projections, which conv ([channels][taps]; inputs: fp32, a slot's last taps - 1 rows of
+// channels at inputs + slot * in_stride, brought up to date by nb_conv_state_update afterwards)
+// convolves and silu activates, else ready; beta: fp32 rows, head h's logit at column beta_col + h;
+// low: fp32 rows with the decay logits (n_heads * d) at decay_col and the gate logits (n_heads * dv)
+// at gate_col; a_log [n_heads], dt_bias [n_heads*d], norm_w [dv]; state: a slot's row at state + slot *
+// state_stride holds [n_heads][d][dv] (key channel, value channel); records: scratch
+// (nb_gated_delta_scratch); o_raw: fp32 scratch [n_rows][n_heads*dv]; out: [n_rows][n_heads*dv].
+NB_EXPORT int nb_gated_delta(const float* qkv, int qkv_stride, int qkv_col, const float* conv, int taps,
+                             float* inputs, int in_stride, const float* beta, int beta_stride,
                              int beta_col, const float* low, int low_stride, int decay_col,
                              int gate_col, const float* a_log, const float* dt_bias,
                              const float* norm_w, float eps, float key_eps, const int* cu_rows,
@@ -622,38 +779,62 @@ NB_EXPORT int nb_gated_delta(const float* qkv, int qkv_stride, const float* beta
   if (n_rows == 0 || n_seqs == 0 || max_q_len == 0) return 0;
   int rc = check_sizes("gated_delta", n_heads, n_kv_heads, d, dv, n_seqs, out_dtype);
   if (rc) return rc;
-  NB_REQUIRE((uintptr_t)records % 16 == 0, NB_ERR_BAD_ARG, "gated_delta: unaligned scratch");
-  const Source src{qkv, qkv_stride, beta, beta_stride, beta_col, low, low_stride, decay_col, gate_col,
-                   a_log, dt_bias};
-  const int vec_in = d % 4 == 0 && qkv_stride % 4 == 0 && low_stride % 4 == 0 && decay_col % 4 == 0 &&
-                     ((uintptr_t)qkv | (uintptr_t)low) % 16 == 0;
+  NB_REQUIRE((uintptr_t)records % 16 == 0 && taps >= 0 && taps <= MAX_FUSED_TAPS && qkv_col >= 0 &&
+                 (taps == 0 || conv != nullptr) && (taps <= 1 || inputs != nullptr),
+             NB_ERR_BAD_ARG, "gated_delta: unaligned scratch or bad taps=%d", taps);
+  const int channels = 2 * n_kv_heads * d + n_heads * dv;
+  const Source src{qkv, qkv_stride, qkv_col, conv, taps, inputs, in_stride, channels, beta, beta_stride,
+                   beta_col, low, low_stride, decay_col, gate_col, a_log, dt_bias};
+  const bool rows16 = qkv_stride % 4 == 0 && qkv_col % 4 == 0 && ((uintptr_t)qkv | (uintptr_t)conv) % 16 == 0;
+  const int vec_in = rows16 && d % 4 == 0 && low_stride % 4 == 0 && decay_col % 4 == 0 && (uintptr_t)low % 16 == 0;
+  const int vec_v = rows16 && dv % 4 == 0 && (2 * n_kv_heads * d) % 4 == 0;
+  const int vec_st = in_stride % 4 == 0 && channels % 4 == 0 && (uintptr_t)inputs % 16 == 0;
   const int vec = dv % 4 == 0 && state_stride % 4 == 0 && ((uintptr_t)state | (uintptr_t)o_raw) % 16 == 0;
   const int blocks = (max_q_len + BLK - 1) / BLK;
   const dim3 grid((blocks + 3) / 4, n_heads, n_seqs);
   const bool long_walk = n_rows > 4 * n_seqs;
-  const int few = n_heads * n_seqs * ((dv + 31) / 32) < 148;     // fewer columns a CTA fill the GPU
-#define NB_GD(CH, LPG, NW)                                                                        \
+#define NB_PREP(DP_, CONV_)                                                                       \
+  NB_CUDA(nb_launch(gated_delta_prepare_kernel<DP_, CONV_>, grid, dim3(128), 0, stream, src,      \
+                    key_eps, cu_rows, seq_slot, records, n_heads, n_kv_heads, d, dv, vec_st,      \
+                    vec_in, vec_v))
+#define NB_WALK(CH, LPG, NC, NW)                                                                  \
+  rc = launch_walk<CH, LPG, NC, NW>(stream, records, cu_rows, seq_slot, state, state_stride, o_raw, \
+                                    n_heads, d, dv, vec, n_seqs, long_walk)
+#define NB_GD(DP_)                                                                                \
   do {                                                                                            \
-    NB_CUDA(nb_launch(gated_delta_prepare_kernel<CH * LPG>, grid, dim3(128), 0, stream, src,      \
-                      key_eps, cu_rows, seq_slot, records, n_heads, n_kv_heads, d, dv, vec_in));  \
+    if (taps == 0) NB_PREP(DP_, 0);                                                               \
+    else if (out_dtype == NB_F32) NB_PREP(DP_, 1);                                                \
+    else NB_PREP(DP_, 2);                                                                         \
     NB_CHECK_LAUNCH("gated_delta_prepare");                                                       \
-    rc = few ? launch_walk<CH, LPG, (NW + 1) / 2>(stream, records, cu_rows, seq_slot, state,      \
-                                                  state_stride, o_raw, n_heads, d, dv, vec,       \
-                                                  n_seqs, long_walk)                              \
-             : launch_walk<CH, LPG, NW>(stream, records, cu_rows, seq_slot, state, state_stride,  \
-                                        o_raw, n_heads, d, dv, vec, n_seqs, long_walk);           \
   } while (0)
-  if (d <= 32) NB_GD(4, 8, 2);
-  else if (d <= 64) NB_GD(4, 16, 4);
-  else if (d <= 128) NB_GD(4, 32, 8);
-  else NB_GD(8, 32, 8);
+  // As measured on prompts of 2 x 1,024 tokens: two columns a lane while the warps are few (a block's
+  // time is one warp's instructions), four where there are heads enough to fill the schedulers.
+  const bool few = (long long)n_heads * n_seqs * ((dv + 31) / 32) <= 148;
+  if (d <= 32) {
+    NB_GD(32);
+    NB_WALK(4, 8, 4, 2);
+  } else if (d <= 64) {
+    NB_GD(64);
+    if (few) NB_WALK(4, 16, 2, 4);
+    else NB_WALK(4, 16, 2, 8);
+  } else if (d <= 128) {
+    NB_GD(128);
+    if (few) NB_WALK(8, 16, 2, 8);
+    else NB_WALK(8, 16, 4, 4);
+  } else {
+    NB_GD(256);
+    NB_WALK(16, 16, 4, 4);
+  }
 #undef NB_GD
+#undef NB_WALK
+#undef NB_PREP
   if (rc) return rc;
   return launch_delta_finish(o_raw, low, low_stride, gate_col, norm_w, 0, eps, row_slot, out, out_dtype,
                              n_heads, dv, n_rows, stream);
 }
 
-// The same for a step of one token per sequence (row cu_rows[s] of sequence s).
+// The same for a step of one token per sequence (row cu_rows[s] of sequence s), its rows ready (qkv from
+// column 0).
 NB_EXPORT int nb_gated_delta_step(const float* qkv, int qkv_stride, const float* beta, int beta_stride,
                                   int beta_col, const float* low, int low_stride, int decay_col,
                                   int gate_col, const float* a_log, const float* dt_bias,
@@ -664,8 +845,8 @@ NB_EXPORT int nb_gated_delta_step(const float* qkv, int qkv_stride, const float*
   if (n_seqs == 0) return 0;
   const int rc = check_sizes("gated_delta_step", n_heads, n_kv_heads, d, dv, n_seqs, out_dtype);
   if (rc) return rc;
-  const Source src{qkv, qkv_stride, beta, beta_stride, beta_col, low, low_stride, decay_col, gate_col,
-                   a_log, dt_bias};
+  const Source src{qkv, qkv_stride, 0, nullptr, 0, nullptr, 0, 2 * n_kv_heads * d + n_heads * dv, beta,
+                   beta_stride, beta_col, low, low_stride, decay_col, gate_col, a_log, dt_bias};
   const int vec = dv % 4 == 0 && state_stride % 4 == 0 && (uintptr_t)state % 16 == 0;
   const int splits = (dv + ST_COLS - 1) / ST_COLS;
   const dim3 grid(splits, n_heads, n_seqs);
@@ -687,3 +868,6 @@ NB_EXPORT int nb_gated_delta_step(const float* qkv, int qkv_stride, const float*
   NB_CHECK_LAUNCH("gated_delta_step");
   return 0;
 }
+
+// The longest convolution that nb_gated_delta takes in (a longer one runs before it).
+NB_EXPORT int nb_gated_delta_max_taps() { return MAX_FUSED_TAPS; }

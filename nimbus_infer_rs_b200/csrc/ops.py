@@ -1081,39 +1081,59 @@ class CudaBackend:
                    layout.n_seqs, n, self._stream())
         self.launches += 1
 
-    def gated_delta(self, qkv, beta, col_beta, low, col_decay, col_gate, a_log, dt_bias, norm, eps,
-                    key_eps, layout, state, n_heads, n_kv_heads, d, dv, out):
+    def gated_delta(self, src, col_qkv, conv, taps, inputs, beta, col_beta, low, col_decay, col_gate,
+                    a_log, dt_bias, norm, eps, key_eps, layout, state, n_heads, n_kv_heads, d, dv, out):
         """The gated delta rule over each sequence's rows in order, from and into the sequences'
-        state rows (``state``: fp32 ``[slots, n_heads * d * dv]``).  ``qkv``: convolved and activated
-        rows ``[q | k | v]`` (``n_kv_heads``, ``n_kv_heads`` and ``n_heads`` heads); ``beta``: rows with
-        the heads' logits at ``col_beta``; ``low``: rows with the decay logits at ``col_decay`` and the
-        output gate's at ``col_gate``; all fp32.  The heads' outputs normed, weighted and gated
-        into ``out``."""
-        for t, nm in ((qkv, "qkv"), (beta, "beta"), (low, "low")):
+        state rows (``state``: fp32 ``[slots, n_heads * d * dv]``).  ``src``: rows with ``[q | k | v]``
+        (``n_kv_heads``, ``n_kv_heads`` and ``n_heads`` heads) from column ``col_qkv``; with ``conv``
+        (``[channels, taps]``) they are projections that a short causal convolution (its last
+        ``taps - 1`` inputs in the state rows ``inputs``, brought up to date) and a silu make ready;
+        ``beta``: rows with the heads' logits at ``col_beta``; ``low``: rows with the decay logits at
+        ``col_decay`` and the output gate's at ``col_gate``; all fp32.  The heads' outputs normed,
+        weighted and gated into ``out``."""
+        for t, nm in ((src, "src"), (beta, "beta"), (low, "low")):
             _check(t, nm, torch.float32, 2)
         _check(out, "out", None, 2)
         n, H, G = layout.n_rows, n_heads, n_kv_heads
-        if out.shape != (n, H * dv) or qkv.shape[0] < n or qkv.shape[1] != 2 * G * d + H * dv or \
+        C = 2 * G * d + H * dv
+        taps = int(taps) if conv is not None else 0
+        if out.shape != (n, H * dv) or src.shape[0] < n or src.shape[1] < col_qkv + C or \
+                (conv is not None and tuple(conv.shape) != (C, taps)) or \
                 beta.shape[0] < n or beta.shape[1] < col_beta + H or low.shape[0] < n or \
                 low.shape[1] < max(col_decay + H * d, col_gate + H * dv) or a_log.numel() != H or \
                 dt_bias.numel() != H * d or norm.numel() != dv:
             raise KernelError("gated_delta: shapes do not agree")
+        one = layout.is_decode and layout.max_q_len == 1
+        if taps > 0 and (one or taps > self.lib.nb_gated_delta_max_taps()):
+            # the convolution on its own: a long one, or a one-token step's (which moves the state
+            # rows' inputs up as it reads them)
+            ready = torch.empty((n, C), device=out.device, dtype=torch.float32)
+            self.conv_act(src, col_qkv, conv, None, taps, ACT_SILU, inputs, layout, ready)
+            src, col_qkv, conv, taps = ready, 0, None, 0
         st = self._state_rows(state, H * d * dv)
-        args = (_ptr(qkv), qkv.shape[1], _ptr(beta), beta.shape[1], col_beta, _ptr(low), low.shape[1],
-                col_decay, col_gate, _ptr(a_log), _ptr(dt_bias), _ptr(norm), float(eps), float(key_eps),
+        ins = self._state_rows(inputs, (taps - 1) * C) if taps > 1 else None
+        args = (_ptr(beta), beta.shape[1], col_beta, _ptr(low), low.shape[1], col_decay, col_gate,
+                _ptr(a_log), _ptr(dt_bias), _ptr(norm), float(eps), float(key_eps),
                 _ptr(layout.cu_rows), _ptr(layout.seq_slot))
-        if layout.is_decode and layout.max_q_len == 1:
-            self._call("nb_gated_delta_step", *args, _ptr(st), st.stride(0), _ptr(out),
-                       dtype_code(out.dtype), H, G, d, dv, layout.n_seqs, self._stream())
+        if one:
+            # (rows that are ready may stand behind other columns)
+            self._call("nb_gated_delta_step", _ptr(src) + 4 * col_qkv, src.shape[1], *args, _ptr(st),
+                       st.stride(0), _ptr(out), dtype_code(out.dtype), H, G, d, dv, layout.n_seqs,
+                       self._stream())
             return
         # what every block of four tokens does to the state, and the outputs before their norm
         records = torch.empty(self.lib.nb_gated_delta_scratch(n, layout.n_seqs, H, d, dv),
                               device=out.device, dtype=torch.float32)
         o_raw = torch.empty((n, H * dv), device=out.device, dtype=torch.float32)
-        self._call("nb_gated_delta", *args, _ptr(layout.row_slot), _ptr(st), st.stride(0),
+        self._call("nb_gated_delta", _ptr(src), src.shape[1], col_qkv, _ptr(conv), taps, _ptr(ins),
+                   ins.stride(0) if ins is not None else 0, *args, _ptr(layout.row_slot), _ptr(st), st.stride(0),
                    _ptr(records), _ptr(o_raw), _ptr(out), dtype_code(out.dtype), H, G, d, dv,
                    layout.n_seqs, layout.max_q_len, n, self._stream())
         self.launches += 2
+        if taps > 1:
+            self._call("nb_conv_state_update", _ptr(src), src.shape[1], col_qkv, taps, _ptr(ins),
+                       ins.stride(0), _ptr(layout.cu_rows), _ptr(layout.seq_slot), C, layout.n_seqs,
+                       self._stream())
 
     # -- short convolutions, capped attention, linear recurrences ------------------------
     @staticmethod

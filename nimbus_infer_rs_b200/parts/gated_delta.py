@@ -3,7 +3,6 @@ from __future__ import annotations
 
 import torch
 
-from ..csrc.ops import ACT_SILU
 from .base import MATRIX, VECTOR, Mixer, ParamSpec, StateRequest, register_part
 from .linear import Linear
 
@@ -25,10 +24,10 @@ class GatedDeltaRule(Mixer):
     ``norm`` (``value_dim`` numbers, shared by the heads) and by ``sigmoid(Wg2 (Wg1 h))``; ``Wout``
     maps the heads side by side back.
 
-    How it runs: one product gives ``[q | k | v | beta logits | Wa1 h | Wg1 h]`` in fp32; the
-    convolution pass keeps its last ``taps - 1`` inputs in the sequence's state row; one small
-    product per head pair maps the two low-rank columns up; the recurrence's kernels do everything
-    else in fp32 and leave the state in the same row.  Nothing grows with the sequence.
+    How it runs: one product gives ``[q | k | v | beta logits | Wa1 h | Wg1 h]`` in fp32; one small
+    product maps the two low-rank columns up; the recurrence's kernels do everything else in fp32,
+    the convolution included, and leave the matrices and the convolution's last ``taps - 1`` inputs
+    in the sequence's state row.  Nothing grows with the sequence.
     """
     graph_safe = True
     can_overwrite = True
@@ -81,14 +80,12 @@ class GatedDeltaRule(Mixer):
         matrices = ctx.state[:, :m]
         inputs = ctx.state[:, m:m + (self.taps - 1) * self.channels]
         fused = self.proj(ctx, h, out_dtype=torch.float32)
-        qkv = torch.empty((n, self.channels), device=dev, dtype=torch.float32)
-        ops.conv_act(fused, 0, self.conv, None, self.taps, ACT_SILU, inputs, lay, qkv)
         low = torch.empty((n, 2 * self.up_width), device=dev, dtype=torch.float32)
         ops.head_linear(fused, self.col_low, self.up, low, lay)
         o = torch.empty((n, self.v_width), device=dev, dtype=act)
-        ops.gated_delta(qkv, fused, self.col_beta, low, 0, self.up_width, self.a_log, self.dt_bias,
-                        self.norm, self.eps, self.key_eps, lay, matrices, self.n_heads,
-                        self.n_kv_heads, self.head_dim, self.value_dim, o)
+        ops.gated_delta(fused, 0, self.conv, self.taps, inputs, fused, self.col_beta, low, 0,
+                        self.up_width, self.a_log, self.dt_bias, self.norm, self.eps, self.key_eps,
+                        lay, matrices, self.n_heads, self.n_kv_heads, self.head_dim, self.value_dim, o)
         if accumulate:
             self.out(ctx, o, residual=residual)
         else:

@@ -315,9 +315,14 @@ class CpuBackend:
             o = o / torch.sqrt((o * o).mean(-1, keepdim=True) + eps)
             out[r] = (o.reshape(hd) * norm_w * g).to(out.dtype)
 
-    def gated_delta(self, qkv, beta, col_beta, low, col_decay, col_gate, a_log, dt_bias, norm, eps,
-                    key_eps, layout, state, n_heads, n_kv_heads, d, dv, out):
+    def gated_delta(self, src, col_qkv, conv, taps, inputs, beta, col_beta, low, col_decay, col_gate,
+                    a_log, dt_bias, norm, eps, key_eps, layout, state, n_heads, n_kv_heads, d, dv, out):
         H, G = n_heads, n_kv_heads
+        qkv = src[:, col_qkv:col_qkv + 2 * G * d + H * dv]
+        if conv is not None:
+            ready = torch.empty(layout.n_rows, qkv.shape[1])
+            self.conv_act(src, col_qkv, conv, None, taps, 3, inputs, layout, ready)
+            qkv = ready
         of = torch.arange(H) // (H // G)
         for r in range(layout.n_rows):
             slot = int(layout.row_slot[r])

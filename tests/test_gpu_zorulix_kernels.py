@@ -338,7 +338,7 @@ def _plain_recurrence(qkv, beta, low, a_log, dt_bias, norm, H, G, d, dv, eps, S=
 def _run(ops, dtype, rows, weights, lay, state, H, G, d, dv, eps):
     qkv, beta, low = (r.to(DEV).contiguous() for r in rows)
     out = torch.full((lay.n_rows, H * dv), 7.0, device=DEV, dtype=ACT[dtype])
-    ops.gated_delta(qkv, beta, 2, low, 3, 3 + H * d, *(w.to(DEV) for w in weights), eps, 1e-6, lay, state,
+    ops.gated_delta(qkv, 0, None, 0, None, beta, 2, low, 3, 3 + H * d, *(w.to(DEV) for w in weights), eps, 1e-6, lay, state,
                     H, G, d, dv, out)
     return out.float().cpu()
 
@@ -450,30 +450,38 @@ def test_unequal_sequences_in_one_batch(ops, dtype, H, G, d, dv):
                 _close(got[i], refs[i][n + step], TOL[dtype], f"{n} tokens and {step + 1}")
 
 
+@pytest.mark.parametrize("H,G,d,dv", [(2, 1, 12, 10), (2, 2, 12, 10), (3, 3, 64, 64), (2, 2, 128, 128),
+                                      (2, 1, 64, 96), (1, 1, 129, 33), (4, 4, 20, 36)])
 @pytest.mark.parametrize("taps", [1, 2, 3, 4, 7])
-def test_convolution_and_recurrence_share_a_state_row(ops, taps):
+def test_convolution_and_recurrence_share_a_state_row(ops, taps, H, G, d, dv):
     """The matrices first, then the convolution's last inputs: a sequence cut anywhere goes on as
-    if it had not been cut, and the row of a slot that is used again starts from zeros."""
-    H, G, d, dv, T, eps = 2, 1, 12, 10, 40, 1e-5
+    if it had not been cut, alone and beside another, and the row of a slot that is used again
+    starts from zeros."""
+    T, eps = 40, 1e-5
     C, n = 2 * G * d + H * dv, H * d * dv
     raw, (_, beta, low), weights = _rnd(T, C, seed=1), _recurrence_inputs(T, H, G, d, dv, 2), _weights(H, d, dv)
     w = _rnd(C, taps, seed=3)
-    qkv = PZ.silu(PZ.causal_conv(raw.double(), w.double()))
-    ref, _ = _plain_recurrence(qkv, beta, low, *weights, H, G, d, dv, eps)
-    cache = SequenceCache({}, {0: StateRequest(n + (taps - 1) * C)}, cache_tokens=64, max_seq_len=64,
-                          dtype=torch.float32, device=torch.device(DEV), n_slots=2)
+    ready = PZ.silu(PZ.causal_conv(raw.double(), w.double()))
+    ref, _ = _plain_recurrence(ready, beta, low, *weights, H, G, d, dv, eps)
+    want = -(-(n + (taps - 1) * C) // 4) * 4
+    cache = SequenceCache({}, {0: StateRequest(want)}, cache_tokens=192, max_seq_len=64,
+                          dtype=torch.float32, device=torch.device(DEV), n_slots=3)
+    src = torch.cat([torch.full((T, 4), 9.0), raw, beta, torch.zeros(T, -(C + beta.shape[1]) % 4)], 1)
     for pieces in ([T], [1] * T, [2, 1, 3, 1, 1, 20, 12]):
-        slot, got, at = cache.alloc_slot(), [], 0
+        slot, beside, got, at = cache.alloc_slot(), cache.alloc_slot(), [], 0
         row = cache.layer_state(0)
         for m in pieces:
-            lay = _layout([(slot, m)], [at])
-            act = torch.empty(m, C, device=DEV)
-            ops.conv_act(raw[at:at + m].to(DEV), 0, w.to(DEV), None, taps, ACT_SILU,
-                         row[:, n:n + (taps - 1) * C], lay, act)
-            out = torch.empty(m, H * dv, device=DEV)
-            ops.gated_delta(act, beta[at:at + m].to(DEV), 2, low[at:at + m].to(DEV), 3, 3 + H * d,
-                            *(x.to(DEV) for x in weights), eps, 1e-6, lay, row[:, :n], H, G, d, dv, out)
-            got.append(out.cpu())
+            # the neighbour: the sequence's first tokens again, one behind in every step
+            lay = _layout([(beside, max(1, m - 1)), (slot, m)], [0, at])
+            both = lambda x: torch.cat([x[:max(1, m - 1)], x[at:at + m]]).to(DEV).contiguous()
+            out = torch.empty(lay.n_rows, H * dv, device=DEV)
+            ops.gated_delta(both(src), 4, w.to(DEV), taps, row[:, n:n + (taps - 1) * C], both(src), 4 + C + 2,
+                            both(low), 3, 3 + H * d, *(x.to(DEV) for x in weights), eps, 1e-6, lay,
+                            row[:, :n], H, G, d, dv, out)
+            got.append(out[max(1, m - 1):].cpu())
             at += m
+        keep = row[slot, n:n + (taps - 1) * C].view(taps - 1, C)
+        assert torch.equal(keep.cpu(), raw[T - taps + 1:])
         cache.free_slot(slot)
+        cache.free_slot(beside)
         _close(torch.cat(got), ref, 5e-5, f"taps {taps}, {pieces[:4]}")
