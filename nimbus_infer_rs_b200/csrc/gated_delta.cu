@@ -8,26 +8,28 @@
 // divided by its root mean square (eps inside the root), times a weight shared by the heads, times
 // sigmoid(gate logits).  Everything is fp32.
 //
-// Prompts.  Four tokens are taken at a time.  With E_(s..t) = the product of g over tokens s+1 .. t
+// Prompts.  Eight tokens are taken at a time.  With E_(s..t) = the product of g over tokens s+1 .. t
 // of the block (per key channel; from the block's start: E_t) and S the state at its start,
 //
 //   u_t = beta_t v_t - (beta_t E_t k_t)^T S - sum_(s<t) A_ts u_s,   A_ts = beta_t sum_i k_ti k_si E_(s..t)i
 //   o_t = (E_t q_t)^T S + sum_(s<=t) B_ts u_s,                     B_ts = sum_i q_ti k_si E_(s..t)i
-//   S  <- diag(E_3) S + sum_s (k_s E_(s..3)) u_s^T
+//   S  <- diag(E_7) S + sum_s (k_s E_(s..7)) u_s^T
 //
-// so the state is read twice and written once per four tokens, the eight dot products of a column
-// with it are independent of one another, and only the four u_t (a few multiply-adds) follow one
+// so the state is read twice and written once per eight tokens, the sixteen dot products of a column
+// with it are independent of one another, and only the eight u_t (a few multiply-adds) follow one
 // another.  Decays are multiplied up, never divided by, so nothing overflows however strong they are.
-//   gated_delta_prepare  a warp per (block of four tokens, head): the short convolution and silu
-//                        of q, k and v (of projected rows, the inputs before the step from the
-//                        state row), then a record: E_3, the four (beta_t E_t k_t), (E_t q_t),
-//                        (k_s E_(s..3)), the numbers A and B, and the four beta_t v_t.  A block's
-//                        missing tokens (a sequence's last block) are tokens with k = q = v = 0, g = 1.
+//   gated_delta_prepare  two warps per (block of eight tokens, head), four tokens each: the short
+//                        convolution and silu of q, k and v (of projected rows, the inputs before
+//                        the step from the state row), then a record: E_7, the eight (beta_t E_t
+//                        k_t), (E_t q_t), (k_s E_(s..7)), the numbers A and B, and the eight beta_t
+//                        v_t.  The first four tokens' part and the second's meet through shared
+//                        memory.  A block's missing tokens (a sequence's last block) are tokens with
+//                        k = q = v = 0, g = 1.
 //   gated_delta_walk     a CTA takes COLS columns of one (sequence, head); the columns are
 //                        independent.  A group of LPG lanes holds NC columns, CH key channels a
 //                        lane, two neighbouring channels in a register pair (packed multiply-adds).
-//                        The 8 NC partial sums of a block (four tokens, NC columns, two products)
-//                        are reduced over the lanes by halving: each lane ends with 8 NC / LPG of
+//                        The 16 NC partial sums of a block (eight tokens, NC columns, two products)
+//                        are reduced over the lanes by halving: each lane ends with 16 NC / LPG of
 //                        them.  Records come through two buffers of asynchronous copies.
 //   delta_finish         norm, weight and gate (the norm needs all of a head's columns).
 // A sequence may be cut into steps anywhere: where blocks begin only changes the rounding.
@@ -40,7 +42,8 @@
 
 namespace {
 
-constexpr int BLK = 4;         // tokens of a block
+constexpr int BLK = 8;         // tokens of a block
+constexpr int HALF = 4;        // ... of a preparing warp
 constexpr int MAX_DIM = 256;
 
 __device__ __forceinline__ float gd_softplus(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
@@ -87,20 +90,22 @@ struct Source {               // where a row's numbers lie
   const float* dt_bias;       // [heads * d]
 };
 
+// A record: E at place 0 (of DP floats), beta E k at 1 .., E q at 1 + BLK .., k E at 1 + 2 BLK .., then A
+// and B (BLK x BLK each) and the values.
 // floats of a record of padded key size DP; dvp: the value size rounded up to a multiple of 4
-__host__ __device__ constexpr int record_head(int DP) { return 13 * DP + 32; }
+__host__ __device__ constexpr int record_head(int DP) { return (3 * BLK + 1) * DP + 2 * BLK * BLK; }
 __host__ __device__ inline int record_floats(int DP, int dvp) { return record_head(DP) + BLK * dvp; }
 
 constexpr int MAX_FUSED_TAPS = 4;
 
-// Four neighbouring channels c .. c+3 (those below `end`) of BLK tokens: y[t] = the ready numbers or
+// Four neighbouring channels c .. c+3 (those below `end`) of HALF tokens: y[t] = the ready numbers or
 // silu of the convolution.  base: the channels' first column in a row; ch0: their first channel.
 // CONV: 0 ready, 1 convolved, 2 convolved with the hardware's exponential and reciprocal in the silu
 // (a bfloat16 run, where projections and their activations are rounded anyway).
 template <int CONV>
 __device__ __forceinline__ void take_channels(const Source& src, const float* in_row, int row0, int row1,
                                               int first, int ch0, int c, int end, bool vec,
-                                              float (&y)[BLK][4]) {
+                                              float (&y)[HALF][4]) {
   auto load4 = [&](const float* p, float (&v)[4]) {
     if (vec && c < end) {
       const float4 f = *reinterpret_cast<const float4*>(p);
@@ -113,14 +118,14 @@ __device__ __forceinline__ void take_channels(const Source& src, const float* in
   const float* col = src.qkv + src.qkv_col + ch0 + c;
   if constexpr (CONV == 0) {
 #pragma unroll
-    for (int t = 0; t < BLK; ++t)
+    for (int t = 0; t < HALF; ++t)
       load4(col + (size_t)(first + t < row1 ? first + t : row0) * src.qkv_stride, y[t]);
   } else {
     // inputs first - 3 .. first + 3; weights with zeros in front up to four taps
-    float x[BLK + MAX_FUSED_TAPS - 1][4], w[MAX_FUSED_TAPS][4];
+    float x[HALF + MAX_FUSED_TAPS - 1][4], w[MAX_FUSED_TAPS][4];
     const int taps = src.taps;
 #pragma unroll
-    for (int i = 0; i < BLK + MAX_FUSED_TAPS - 1; ++i) {
+    for (int i = 0; i < HALF + MAX_FUSED_TAPS - 1; ++i) {
       const int r = first - (MAX_FUSED_TAPS - 1) + i;
       const int back = row0 - r;                 // rows before the step's first: 1 is the newest
       if (back <= 0) load4(col + (size_t)(r < row1 ? r : row0) * src.qkv_stride, x[i]);
@@ -144,7 +149,7 @@ __device__ __forceinline__ void take_channels(const Source& src, const float* in
         }
     }
 #pragma unroll
-    for (int t = 0; t < BLK; ++t)
+    for (int t = 0; t < HALF; ++t)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         float v = 0.0f;
@@ -155,7 +160,7 @@ __device__ __forceinline__ void take_channels(const Source& src, const float* in
   }
 }
 
-// A sequence's blocks start at record cu_rows[seq] / 4 + seq, so that no two sequences overlap.
+// A sequence's blocks start at record cu_rows[seq] / BLK + seq, so that no two sequences overlap.
 template <int DP, int CONV>
 __global__ void __launch_bounds__(128)
 gated_delta_prepare_kernel(Source src, float key_eps, const int* cu_rows, const int* seq_slot,
@@ -164,11 +169,15 @@ gated_delta_prepare_kernel(Source src, float key_eps, const int* cu_rows, const 
   nb_grid_dependency_wait();
   nb_launch_dependents();
   constexpr int KIT = (DP + 127) / 128;             // quads of channels a lane holds
-  const int seq = blockIdx.z, h = blockIdx.y, lane = threadIdx.x & 31;
-  const int blk = blockIdx.x * 4 + (threadIdx.x >> 5);
-  const int row0 = cu_rows[seq], row1 = cu_rows[seq + 1];
-  const int first = row0 + blk * BLK, slot = seq_slot[seq];
-  if (slot < 0 || first >= row1) return;
+  constexpr int N = KIT * 4;
+  __shared__ __align__(16) float kh_s[2][HALF][DP], e_s[2][2][DP];
+  const int seq = blockIdx.z, h = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int pair = warp >> 1, part = warp & 1;      // the CTA's block, and which of its halves
+  const int blk = blockIdx.x * 2 + pair;
+  const int row0 = cu_rows[seq], row1 = cu_rows[seq + 1], slot = seq_slot[seq];
+  if (slot < 0 || row0 + (int)blockIdx.x * 2 * BLK >= row1) return;      // the whole CTA
+  const bool there = row0 + blk * BLK < row1;
+  const int first = row0 + blk * BLK + part * HALF; // of this warp's tokens
   const int g = h / (n_heads / n_kv_heads);
   const int dvp = (dv + 3) & ~3;
   float* rec = records + ((size_t)(row0 / BLK + seq + blk) * n_heads + h) * record_floats(DP, dvp);
@@ -176,125 +185,201 @@ gated_delta_prepare_kernel(Source src, float key_eps, const int* cu_rows, const 
   const float rate = expf(src.a_log[h]);
   const float q_scale = 1.0f / sqrtf((float)d);
   // 16-byte loads of the rows; near the step's start also of the state row
-  const bool vec_q = vec_in && (!CONV || vec || blk > 0);
+  const bool inner = !CONV || vec || blk > 0 || part > 0;
+  const bool vec_q = vec_in && inner;
+  auto place = [&](int p, int j) { return rec + p * DP + (j * 32 + lane) * 4; };
+  auto has = [&](int j) { return (j * 32 + lane) * 4 < DP; };
+  auto store = [&](int p, const float (&v)[N]) {
+#pragma unroll
+    for (int j = 0; j < KIT; ++j)
+      if (has(j))
+        *reinterpret_cast<float4*>(place(p, j)) = make_float4(v[j * 4], v[j * 4 + 1], v[j * 4 + 2], v[j * 4 + 3]);
+  };
+  auto put = [&](float* at, const float (&v)[N]) {        // into a row of shared memory
+#pragma unroll
+    for (int j = 0; j < KIT; ++j)
+      if (has(j))
+        *reinterpret_cast<float4*>(at + (j * 32 + lane) * 4) =
+            make_float4(v[j * 4], v[j * 4 + 1], v[j * 4 + 2], v[j * 4 + 3]);
+  };
+  auto take = [&](const float* at, float (&v)[N]) {
+#pragma unroll
+    for (int j = 0; j < KIT; ++j) {
+      const float4 f = has(j) ? *reinterpret_cast<const float4*>(at + (j * 32 + lane) * 4)
+                              : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+      v[j * 4] = f.x; v[j * 4 + 1] = f.y; v[j * 4 + 2] = f.z; v[j * 4 + 3] = f.w;
+    }
+  };
 
-  float k[BLK][KIT * 4], q[BLK][KIT * 4], w[BLK][KIT * 4], beta[BLK];
-#pragma unroll
-  for (int j = 0; j < KIT; ++j) {
-    const int c = (j * 32 + lane) * 4;
-    float y[BLK][4];
-    take_channels<CONV>(src, in_row, row0, row1, first, g * d, c, d, vec_q, y);
-#pragma unroll
-    for (int t = 0; t < BLK; ++t)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) q[t][j * 4 + e] = y[t][e];
-    take_channels<CONV>(src, in_row, row0, row1, first, (n_kv_heads + g) * d, c, d, vec_q, y);
-#pragma unroll
-    for (int t = 0; t < BLK; ++t) {
-      const int r = first + t < row1 ? first + t : row0;
-      const float* dl = src.low + (size_t)r * src.low_stride + src.decay_col + h * d + c;
-#pragma unroll
-      for (int e = 0; e < 4; ++e) k[t][j * 4 + e] = y[t][e];
-      if (vec_in && c < d) {
-        const float4 f = *reinterpret_cast<const float4*>(dl);
-        w[t][j * 4] = f.x; w[t][j * 4 + 1] = f.y; w[t][j * 4 + 2] = f.z; w[t][j * 4 + 3] = f.w;
-      } else {
-#pragma unroll
-        for (int e = 0; e < 4; ++e) w[t][j * 4 + e] = c + e < d ? dl[e] : 0.0f;
-      }
-    }
-  }
-#pragma unroll
-  for (int t = 0; t < BLK; ++t)
-    beta[t] = first + t < row1
-                  ? nb_sigmoid(src.beta[(size_t)(first + t) * src.beta_stride + src.beta_col + h]) : 0.0f;
-  // unit vectors and decays
-  float ss[2 * BLK];
-#pragma unroll
-  for (int t = 0; t < BLK; ++t) {
-    ss[t] = ss[BLK + t] = 0.0f;
-#pragma unroll
-    for (int i = 0; i < KIT * 4; ++i) {
-      ss[t] = fmaf(k[t][i], k[t][i], ss[t]);
-      ss[BLK + t] = fmaf(q[t][i], q[t][i], ss[BLK + t]);
-    }
-  }
-#pragma unroll
-  for (int i = 0; i < 2 * BLK; ++i) ss[i] = nb_warp_sum(ss[i]);
-#pragma unroll
-  for (int t = 0; t < BLK; ++t) {
-    const bool live = first + t < row1;
-    const float ik = live ? 1.0f / sqrtf(ss[t] + key_eps) : 0.0f;
-    const float iq = live ? q_scale / sqrtf(ss[BLK + t] + key_eps) : 0.0f;
-#pragma unroll
-    for (int i = 0; i < KIT * 4; ++i) {
-      const int c = ((i >> 2) * 32 + lane) * 4 + (i & 3);
-      k[t][i] *= ik;
-      q[t][i] *= iq;
-      w[t][i] = (live && c < d) ? expf(-rate * gd_softplus(w[t][i] + src.dt_bias[h * d + c])) : 1.0f;
-    }
-  }
-  auto store = [&](int place, const float (&v)[KIT * 4]) {
+  float k[HALF][N], q[HALF][N], w[HALF][N], beta[HALF], ab[16];
+  if (there) {
 #pragma unroll
     for (int j = 0; j < KIT; ++j) {
       const int c = (j * 32 + lane) * 4;
-      if (c < DP)
-        *reinterpret_cast<float4*>(rec + place * DP + c) =
-            make_float4(v[j * 4], v[j * 4 + 1], v[j * 4 + 2], v[j * 4 + 3]);
-    }
-  };
-  // the numbers A (six of them) and B (ten), and k_s E_(s..3)
-  float ab[16];
+      float y[HALF][4];
+      take_channels<CONV>(src, in_row, row0, row1, first, g * d, c, d, vec_q, y);
 #pragma unroll
-  for (int s = 0; s < BLK; ++s) {
-    float kd[KIT * 4];
+      for (int t = 0; t < HALF; ++t)
 #pragma unroll
-    for (int i = 0; i < KIT * 4; ++i) kd[i] = k[s][i];
+        for (int e = 0; e < 4; ++e) q[t][j * 4 + e] = y[t][e];
+      take_channels<CONV>(src, in_row, row0, row1, first, (n_kv_heads + g) * d, c, d, vec_q, y);
 #pragma unroll
-    for (int t = s; t < BLK; ++t) {
-      float a = 0.0f, b = 0.0f;
+      for (int t = 0; t < HALF; ++t) {
+        const int r = first + t < row1 ? first + t : row0;
+        const float* dl = src.low + (size_t)r * src.low_stride + src.decay_col + h * d + c;
 #pragma unroll
-      for (int i = 0; i < KIT * 4; ++i) {
-        if (t > s) kd[i] *= w[t][i];
-        a = fmaf(k[t][i], kd[i], a);
-        b = fmaf(q[t][i], kd[i], b);
+        for (int e = 0; e < 4; ++e) k[t][j * 4 + e] = y[t][e];
+        if (vec_in && c < d) {
+          const float4 f = *reinterpret_cast<const float4*>(dl);
+          w[t][j * 4] = f.x; w[t][j * 4 + 1] = f.y; w[t][j * 4 + 2] = f.z; w[t][j * 4 + 3] = f.w;
+        } else {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) w[t][j * 4 + e] = c + e < d ? dl[e] : 0.0f;
+        }
       }
-      if (t > s) ab[t * (t - 1) / 2 + s] = a;
-      ab[6 + t * (t + 1) / 2 + s] = b;
     }
-    store(9 + s, kd);
+#pragma unroll
+    for (int t = 0; t < HALF; ++t)
+      beta[t] = first + t < row1
+                    ? nb_sigmoid(src.beta[(size_t)(first + t) * src.beta_stride + src.beta_col + h]) : 0.0f;
+    // unit vectors and decays
+    float ss[2 * HALF];
+#pragma unroll
+    for (int t = 0; t < HALF; ++t) {
+      ss[t] = ss[HALF + t] = 0.0f;
+#pragma unroll
+      for (int i = 0; i < N; ++i) {
+        ss[t] = fmaf(k[t][i], k[t][i], ss[t]);
+        ss[HALF + t] = fmaf(q[t][i], q[t][i], ss[HALF + t]);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < 2 * HALF; ++i) ss[i] = nb_warp_sum(ss[i]);
+#pragma unroll
+    for (int t = 0; t < HALF; ++t) {
+      const bool live = first + t < row1;
+      const float ik = live ? 1.0f / sqrtf(ss[t] + key_eps) : 0.0f;
+      const float iq = live ? q_scale / sqrtf(ss[HALF + t] + key_eps) : 0.0f;
+#pragma unroll
+      for (int i = 0; i < N; ++i) {
+        const int c = ((i >> 2) * 32 + lane) * 4 + (i & 3);
+        k[t][i] *= ik;
+        q[t][i] *= iq;
+        w[t][i] = (live && c < d) ? expf(-rate * gd_softplus(w[t][i] + src.dt_bias[h * d + c])) : 1.0f;
+      }
+    }
+    // A (six numbers) and B (ten) among this half's tokens, and k_s decayed to the half's end
+#pragma unroll
+    for (int s = 0; s < HALF; ++s) {
+      float kd[N];
+#pragma unroll
+      for (int i = 0; i < N; ++i) kd[i] = k[s][i];
+#pragma unroll
+      for (int t = s; t < HALF; ++t) {
+        float a = 0.0f, b = 0.0f;
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+          if (t > s) kd[i] *= w[t][i];
+          a = fmaf(k[t][i], kd[i], a);
+          b = fmaf(q[t][i], kd[i], b);
+        }
+        if (t > s) ab[t * (t - 1) / 2 + s] = a;
+        ab[6 + t * (t + 1) / 2 + s] = b;
+      }
+      if (part == 0) put(kh_s[pair][s], kd);
+      else store(1 + 2 * BLK + HALF + s, kd);
+    }
+    reduce_by_halving<16, 32, 1>(ab, lane);           // lane l holds number l / 2
+    // beta_t E_t k_t and E_t q_t from the half's start
+#pragma unroll
+    for (int t = 0; t < HALF; ++t)
+#pragma unroll
+      for (int i = 0; i < N; ++i) {
+        if (t > 0) w[t][i] *= w[t - 1][i];
+        k[t][i] *= beta[t] * w[t][i];
+        q[t][i] *= w[t][i];
+      }
+    put(e_s[pair][part], w[HALF - 1]);
   }
-  reduce_by_halving<16, 32, 1>(ab, lane);           // lane l holds number l / 2
+  __syncthreads();
+  if (!there) return;
+  // a row of A and of B: slot `lane` is row t of the half, column s of the block
+  float across[32];
+  if (part == 0) {
+    float e2[N], e[N];
+    take(e_s[pair][1], e2);
+#pragma unroll
+    for (int s = 0; s < HALF; ++s) {
+      float kd[N];
+      take(kh_s[pair][s], kd);
+#pragma unroll
+      for (int i = 0; i < N; ++i) kd[i] *= e2[i];
+      store(1 + 2 * BLK + s, kd);
+      store(1 + s, k[s]);
+      store(1 + BLK + s, q[s]);
+    }
+#pragma unroll
+    for (int i = 0; i < N; ++i) e[i] = w[HALF - 1][i] * e2[i];
+    store(0, e);
+  } else {
+    float e1[N];
+    take(e_s[pair][0], e1);
+#pragma unroll
+    for (int s = 0; s < HALF; ++s) {
+      float kd[N];
+      take(kh_s[pair][s], kd);
+#pragma unroll
+      for (int t = 0; t < HALF; ++t) {
+        float a = 0.0f, b = 0.0f;
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+          a = fmaf(k[t][i], kd[i], a);
+          b = fmaf(q[t][i], kd[i], b);
+        }
+        across[t * HALF + s] = a;
+        across[16 + t * HALF + s] = b;
+      }
+    }
+    reduce_by_halving<32, 32, 1>(across, lane);      // lane l holds number l
+#pragma unroll
+    for (int t = 0; t < HALF; ++t) {
+#pragma unroll
+      for (int i = 0; i < N; ++i) {
+        k[t][i] *= e1[i];
+        q[t][i] *= e1[i];
+      }
+      store(1 + HALF + t, k[t]);
+      store(1 + BLK + HALF + t, q[t]);
+    }
+  }
   {
-    const int t = (lane & 15) >> 2, s = lane & 3;   // slot `lane`: A (0..15), B (16..31), row t, column s
-    const bool is_b = lane >= 16, there = is_b ? s <= t : s < t;
-    const int idx = is_b ? 6 + t * (t + 1) / 2 + s : t * (t - 1) / 2 + s;
-    float v = __shfl_sync(0xffffffffu, ab[0], there ? 2 * idx : 0);
+    const int t = lane >> 3, col = lane & 7, s = col - part * HALF;     // s: within the half
     const float bt = t == 0 ? beta[0] : t == 1 ? beta[1] : t == 2 ? beta[2] : beta[3];
-    rec[13 * DP + lane] = there ? (is_b ? v : v * bt) : 0.0f;
-  }
-  // beta_t E_t k_t, E_t q_t, E_3
-#pragma unroll
-  for (int t = 0; t < BLK; ++t) {
-    float kt[KIT * 4], qt[KIT * 4];
-#pragma unroll
-    for (int i = 0; i < KIT * 4; ++i) {
-      if (t > 0) w[t][i] *= w[t - 1][i];
-      kt[i] = beta[t] * k[t][i] * w[t][i];
-      qt[i] = q[t][i] * w[t][i];
+    const bool in_a = s >= 0 && s < t, in_b = s >= 0 && s <= t && s < HALF;
+    float a = __shfl_sync(0xffffffffu, ab[0], in_a ? 2 * (t * (t - 1) / 2 + s) : 0) * bt;
+    float b = __shfl_sync(0xffffffffu, ab[0], in_b ? 2 * (6 + t * (t + 1) / 2 + s) : 0);
+    if (!in_a) a = 0.0f;
+    if (!in_b) b = 0.0f;
+    if (part == 1) {
+      const float xa = __shfl_sync(0xffffffffu, across[0], col < HALF ? t * HALF + col : 0);
+      const float xb = __shfl_sync(0xffffffffu, across[0], col < HALF ? 16 + t * HALF + col : 0);
+      if (col < HALF) {
+        a = xa;
+        b = xb;
+      }
     }
-    store(1 + t, kt);
-    store(5 + t, qt);
+    float* at = rec + (3 * BLK + 1) * DP + (part * HALF + t) * BLK + col;
+    at[0] = a;
+    at[BLK * BLK] = b;
   }
-  store(0, w[BLK - 1]);
   // beta_t v_t
-  float* vd = rec + record_head(DP);
+  float* vd = rec + record_head(DP) + part * HALF * dvp;
   for (int c = lane * 4; c < dvp; c += 128) {
-    float y[BLK][4];
+    float y[HALF][4];
     take_channels<CONV>(src, in_row, row0, row1, first, 2 * n_kv_heads * d + h * dv, c, dv,
-                        vec_v && (!CONV || vec || blk > 0), y);
+                        vec_v && inner, y);
 #pragma unroll
-    for (int t = 0; t < BLK; ++t) {
+    for (int t = 0; t < HALF; ++t) {
       const float b = beta[t];                     // zero for a missing token
       *reinterpret_cast<float4*>(vd + t * dvp + c) =
           make_float4(b * y[t][0], b * y[t][1], b * y[t][2], b * y[t][3]);
@@ -350,7 +435,7 @@ struct Walk {
   static constexpr int GROUPS = NW * GPW;
   static constexpr int COLS = NC * GROUPS;
   static constexpr int V = 2 * BLK * NC;                         // sums of a block and group
-  static constexpr int SB = DP > 128 ? 2 : 4;                    // blocks a buffer holds
+  static constexpr int SB = DP > 128 ? 1 : 2;                    // blocks a buffer holds
   static constexpr int BUF = SB * (record_head(DP) + BLK * COLS);  // floats of a buffer
   static constexpr int SMEM = (2 * BUF + 2 * GROUPS * V) * 4;
 };
@@ -386,7 +471,7 @@ gated_delta_walk_kernel(const float* records, const int* cu_rows, const int* seq
     for (int b = 0; b < nb; ++b) {
       const float* rec = recs + (size_t)(b0 + b) * rec_step;
       for (int i = tid; i < HEAD / 4; i += THREADS) cp_async16(dst + b * HEAD + i * 4, rec + i * 4);
-      for (int i = tid; i < COLS; i += THREADS) {   // BLK rows of COLS / 4 pieces
+      for (int i = tid; i < BLK * COLS / 4; i += THREADS) {
         const int t = i / (COLS / 4), c = (i % (COLS / 4)) * 4;
         if (col0 + c < dvp)
           cp_async16(dst + SB * HEAD + (b * BLK + t) * COLS + c, rec + HEAD + t * dvp + col0 + c);
@@ -435,31 +520,26 @@ gated_delta_walk_kernel(const float* records, const int* cu_rows, const int* seq
     const int nb = min(SB, n_blocks - b0);
     for (int b = 0; b < nb; ++b, head += HEAD, vals += BLK * COLS) {
       // (beta E k)_t . S_c at t NC + c,  (E q)_t . S_c at V / 2 + t NC + c
-      f32x2 acc[V];
-#pragma unroll
-      for (int i = 0; i < V; ++i) acc[i] = 0ull;
-#pragma unroll
-      for (int g = 0; g < CH / 4; ++g) {
-#pragma unroll
-        for (int t = 0; t < BLK; ++t) {
-          const ulonglong2 kk = *reinterpret_cast<const ulonglong2*>(head + (1 + t) * DP + (g * LPG + q) * 4);
-          const ulonglong2 qq = *reinterpret_cast<const ulonglong2*>(head + (5 + t) * DP + (g * LPG + q) * 4);
-#pragma unroll
-          for (int c = 0; c < NC; ++c) {
-            f32x2& r = acc[t * NC + c];
-            f32x2& o = acc[V / 2 + t * NC + c];
-            r = fma2(kk.x, S[2 * g][c], r);
-            r = fma2(kk.y, S[2 * g + 1][c], r);
-            o = fma2(qq.x, S[2 * g][c], o);
-            o = fma2(qq.y, S[2 * g + 1][c], o);
-          }
-        }
-      }
       float p[V];
 #pragma unroll
-      for (int i = 0; i < V; ++i) {
-        const float2 f = unpair(acc[i]);
-        p[i] = f.x + f.y;
+      for (int t = 0; t < 2 * BLK; ++t) {           // the places 1 .. 2 BLK of the record
+        f32x2 acc[NC];
+#pragma unroll
+        for (int c = 0; c < NC; ++c) acc[c] = 0ull;
+#pragma unroll
+        for (int g = 0; g < CH / 4; ++g) {
+          const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(head + (1 + t) * DP + (g * LPG + q) * 4);
+#pragma unroll
+          for (int c = 0; c < NC; ++c) {
+            acc[c] = fma2(x.x, S[2 * g][c], acc[c]);
+            acc[c] = fma2(x.y, S[2 * g + 1][c], acc[c]);
+          }
+        }
+#pragma unroll
+        for (int c = 0; c < NC; ++c) {
+          const float2 f = unpair(acc[c]);
+          p[t * NC + c] = f.x + f.y;
+        }
       }
       reduce_by_halving<V, LPG, GPW>(p, q);
       float* mine = red + (parity * W::GROUPS + group) * V;
@@ -467,21 +547,25 @@ gated_delta_walk_kernel(const float* records, const int* cu_rows, const int* seq
 #pragma unroll
       for (int i = 0; i < V / LPG; ++i) mine[q * (V / LPG) + i] = p[i];
       __syncwarp();
-      // the four u
+      // the eight u
       float u[BLK][NC];
+      const float* amat = head + (3 * BLK + 1) * DP;
 #pragma unroll
       for (int t = 0; t < BLK; ++t) {
         float r[NC];
         load_cols<NC>(mine + t * NC, r);
         load_cols<NC>(vals + t * COLS, u[t]);
-        float4 a = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-        if (t > 0) a = *reinterpret_cast<const float4*>(head + 13 * DP + 4 * t);
+        float a[BLK];
+#pragma unroll
+        for (int s4 = 0; s4 < (t + 3) / 4; ++s4) {
+          const float4 f = *reinterpret_cast<const float4*>(amat + t * BLK + s4 * 4);
+          a[s4 * 4] = f.x; a[s4 * 4 + 1] = f.y; a[s4 * 4 + 2] = f.z; a[s4 * 4 + 3] = f.w;
+        }
 #pragma unroll
         for (int c = 0; c < NC; ++c) {
           u[t][c] -= r[c];
-          if (t > 0) u[t][c] = fmaf(-a.x, u[0][c], u[t][c]);
-          if (t > 1) u[t][c] = fmaf(-a.y, u[1][c], u[t][c]);
-          if (t > 2) u[t][c] = fmaf(-a.z, u[2][c], u[t][c]);
+#pragma unroll
+          for (int s2 = 0; s2 < t; ++s2) u[t][c] = fmaf(-a[s2], u[s2][c], u[t][c]);
         }
       }
       // the state
@@ -500,7 +584,7 @@ gated_delta_walk_kernel(const float* records, const int* cu_rows, const int* seq
         }
 #pragma unroll
         for (int t = 0; t < BLK; ++t) {
-          const ulonglong2 kk = *reinterpret_cast<const ulonglong2*>(head + (9 + t) * DP + (g * LPG + q) * 4);
+          const ulonglong2 kk = *reinterpret_cast<const ulonglong2*>(head + (1 + 2 * BLK + t) * DP + (g * LPG + q) * 4);
 #pragma unroll
           for (int c = 0; c < NC; ++c) {
             S[2 * g][c] = fma2(kk.x, uu[t][c], S[2 * g][c]);
@@ -512,10 +596,14 @@ gated_delta_walk_kernel(const float* records, const int* cu_rows, const int* seq
       if (token < o_rows) {
         float o[NC];
         load_cols<NC>(mine + V / 2 + q * NC, o);
-        const float4 bb = *reinterpret_cast<const float4*>(head + 13 * DP + 16 + 4 * q);
 #pragma unroll
-        for (int c = 0; c < NC; ++c)
-          o[c] = fmaf(bb.x, u[0][c], fmaf(bb.y, u[1][c], fmaf(bb.z, u[2][c], fmaf(bb.w, u[3][c], o[c]))));
+        for (int s4 = 0; s4 < BLK / 4; ++s4) {
+          const float4 f = *reinterpret_cast<const float4*>(amat + BLK * BLK + q * BLK + s4 * 4);
+#pragma unroll
+          for (int c = 0; c < NC; ++c)
+            o[c] = fmaf(f.x, u[s4 * 4][c], fmaf(f.y, u[s4 * 4 + 1][c],
+                   fmaf(f.z, u[s4 * 4 + 2][c], fmaf(f.w, u[s4 * 4 + 3][c], o[c]))));
+        }
         if (vec) {
           store_cols<NC>(o_at, o);
         } else {
@@ -791,7 +879,7 @@ NB_EXPORT int nb_gated_delta(const float* qkv, int qkv_stride, int qkv_col, cons
   const int vec_st = in_stride % 4 == 0 && channels % 4 == 0 && (uintptr_t)inputs % 16 == 0;
   const int vec = dv % 4 == 0 && state_stride % 4 == 0 && ((uintptr_t)state | (uintptr_t)o_raw) % 16 == 0;
   const int blocks = (max_q_len + BLK - 1) / BLK;
-  const dim3 grid((blocks + 3) / 4, n_heads, n_seqs);
+  const dim3 grid((blocks + 1) / 2, n_heads, n_seqs);
   const bool long_walk = n_rows > 4 * n_seqs;
 #define NB_PREP(DP_, CONV_)                                                                       \
   NB_CUDA(nb_launch(gated_delta_prepare_kernel<DP_, CONV_>, grid, dim3(128), 0, stream, src,      \
@@ -807,23 +895,22 @@ NB_EXPORT int nb_gated_delta(const float* qkv, int qkv_stride, int qkv_col, cons
     else NB_PREP(DP_, 2);                                                                         \
     NB_CHECK_LAUNCH("gated_delta_prepare");                                                       \
   } while (0)
-  // As measured on prompts of 2 x 1,024 tokens: two columns a lane while the warps are few (a block's
-  // time is one warp's instructions), four where there are heads enough to fill the schedulers.
+  // As measured on prompts of 2 x 1,024 tokens: two columns a lane (a block's time is one warp's
+  // instructions), four for heads of up to 64 where there are enough of them to fill the schedulers.
   const bool few = (long long)n_heads * n_seqs * ((dv + 31) / 32) <= 148;
   if (d <= 32) {
     NB_GD(32);
-    NB_WALK(4, 8, 4, 2);
+    NB_WALK(4, 8, 2, 4);
   } else if (d <= 64) {
     NB_GD(64);
     if (few) NB_WALK(4, 16, 2, 4);
-    else NB_WALK(4, 16, 2, 8);
+    else NB_WALK(4, 16, 4, 4);
   } else if (d <= 128) {
     NB_GD(128);
-    if (few) NB_WALK(8, 16, 2, 8);
-    else NB_WALK(8, 16, 4, 4);
+    NB_WALK(8, 16, 2, 8);
   } else {
     NB_GD(256);
-    NB_WALK(16, 16, 4, 4);
+    NB_WALK(16, 16, 2, 8);
   }
 #undef NB_GD
 #undef NB_WALK
