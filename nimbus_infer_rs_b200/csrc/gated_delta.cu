@@ -35,8 +35,10 @@
 // A sequence may be cut into steps anywhere: where blocks begin only changes the rounding.
 //
 // One-token steps.  gated_delta_step: a CTA per (sequence, head, 32 columns), the CTAs of a head in a
-// thread-block cluster that adds up the head's sum of squares through shared memory; the state is
-// fetched before the wait on the kernel in front (which never writes it), read and written once.
+// thread-block cluster that adds up the head's sum of squares through shared memory, or, where there
+// are heads enough to fill the GPU, a CTA per 128 columns.  The state is fetched before the wait on
+// the kernel in front (which never writes it), read and written once; both products with it are
+// taken of the decayed state (S_t^T q = S'^T q + (k . q) u), so their sums meet in one exchange.
 #include "delta_common.cuh"
 #include "attention_common.cuh"
 
@@ -641,37 +643,40 @@ gated_delta_walk_kernel(const float* records, const int* cu_rows, const int* seq
   }
 }
 
-// One token per sequence.  Thread: four neighbouring columns (cq) of the key channels rg, rg + 32, ...
-constexpr int ST_THREADS = 256, ST_COLS = 32;
+// One token per sequence.  COLS columns a CTA; thread: four neighbouring ones (cq) of the key channels
+// rg, rg + RG, ...
+constexpr int ST_THREADS = 256;
 
-template <int NV, typename TOut>
-__global__ void __launch_bounds__(ST_THREADS)
+template <int NV, int COLS, typename TOut>
+__global__ void __launch_bounds__(ST_THREADS, COLS == 128 ? 2 : 1)
 gated_delta_step_kernel(Source src, float key_eps, const float* __restrict__ norm_w, float eps,
                         const int* cu_rows, const int* seq_slot, float* state, int state_stride,
                         TOut* out, int n_heads, int n_kv_heads, int d, int dv, int vec) {
-  __shared__ float k_s[NV * 32], q_s[NV * 32], w_s[NV * 32];
-  __shared__ __align__(16) float part[ST_THREADS / 32][ST_COLS];
-  __shared__ float red[2][8], square[8];
+  constexpr int CQ = COLS / 4, RG = ST_THREADS / CQ, NW = ST_THREADS / 32;
+  static_assert(CQ == 8 || CQ == 32, "a warp covers whole rows of columns");
+  __shared__ float k_s[NV * RG], q_s[NV * RG], w_s[NV * RG];
+  __shared__ __align__(16) float part[2][NW][COLS];
+  __shared__ float red[3][NW], square[8];
   const int split = blockIdx.x, h = blockIdx.y, seq = blockIdx.z, tid = threadIdx.x;
   const int lane = tid & 31, warp = tid >> 5;
-  const int n_splits = gridDim.x;
+  const int n_splits = gridDim.x;                   // the cluster
   const int r = cu_rows[seq], slot = cu_rows[seq + 1] > r ? seq_slot[seq] : -1;
   const int hv = n_heads * dv;
   if (slot < 0) {              // the whole cluster leaves
     nb_grid_dependency_wait();
     nb_launch_dependents();
-    const int c = split * ST_COLS + tid;
-    if (cu_rows[seq + 1] > r && tid < ST_COLS && c < dv)
+    const int c = split * COLS + tid;
+    if (cu_rows[seq + 1] > r && tid < COLS && c < dv)
       out[(size_t)r * hv + h * dv + c] = nb_from_f32<TOut>(0.0f);
     return;
   }
-  const int cq = tid & 7, rg = tid >> 3, col = split * ST_COLS + cq * 4;
+  const int cq = tid % CQ, rg = tid / CQ, col = split * COLS + cq * 4;
   const int g = h / (n_heads / n_kv_heads);
   float* st = state + (size_t)slot * state_stride + (size_t)h * d * dv;
   float S[NV][4];
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
-    const int k = rg + 32 * i;
+    const int k = rg + RG * i;
     S[i][0] = S[i][1] = S[i][2] = S[i][3] = 0.0f;
     if (k >= d || col >= dv) continue;
     if (vec) {
@@ -686,121 +691,135 @@ gated_delta_step_kernel(Source src, float key_eps, const float* __restrict__ nor
   nb_grid_dependency_wait();
   // every CTA of the cluster says that it runs; the matching wait stands in front of the first
   // store into another CTA's shared memory
-  asm volatile("barrier.cluster.arrive.relaxed.aligned;\n" ::: "memory");
+  if (n_splits > 1) asm volatile("barrier.cluster.arrive.relaxed.aligned;\n" ::: "memory");
 
   const float* row = src.qkv + (size_t)r * src.qkv_stride + src.qkv_col;
-  float v4[4];
+  const float* low = src.low + (size_t)r * src.low_stride;
+  float v4[4], gate[4];
 #pragma unroll
-  for (int j = 0; j < 4; ++j) v4[j] = col + j < dv ? row[2 * n_kv_heads * d + h * dv + col + j] : 0.0f;
+  for (int j = 0; j < 4; ++j) {
+    const bool in = col + j < dv;
+    v4[j] = in ? row[2 * n_kv_heads * d + h * dv + col + j] : 0.0f;
+    gate[j] = (in && tid < CQ) ? low[src.gate_col + h * dv + col + j] : 0.0f;
+  }
   const float beta = nb_sigmoid(src.beta[(size_t)r * src.beta_stride + src.beta_col + h]);
-  const float gate = (tid < ST_COLS && split * ST_COLS + tid < dv)
-                         ? src.low[(size_t)r * src.low_stride + src.gate_col + h * dv + split * ST_COLS + tid]
-                         : 0.0f;
   float kx = 0.0f, qx = 0.0f, wx = 0.0f;
   if (tid < d) {
     kx = row[(n_kv_heads + g) * d + tid];
     qx = row[g * d + tid];
-    wx = expf(-expf(src.a_log[h]) *
-              gd_softplus(src.low[(size_t)r * src.low_stride + src.decay_col + h * d + tid] +
-                          src.dt_bias[h * d + tid]));
+    wx = expf(-expf(src.a_log[h]) * gd_softplus(low[src.decay_col + h * d + tid] + src.dt_bias[h * d + tid]));
   }
-  const float sk = nb_warp_sum(kx * kx), sq = nb_warp_sum(qx * qx);
+  const float sk = nb_warp_sum(kx * kx), sq = nb_warp_sum(qx * qx), skq = nb_warp_sum(kx * qx);
   if (lane == 0) {
     red[0][warp] = sk;
     red[1][warp] = sq;
+    red[2][warp] = skq;
   }
   __syncthreads();
-  float tk = 0.0f, tq = 0.0f;
+  float tk = 0.0f, tq = 0.0f, kq = 0.0f;
 #pragma unroll
-  for (int i = 0; i < 8; ++i) {
+  for (int i = 0; i < NW; ++i) {
     tk += red[0][i];
     tq += red[1][i];
+    kq += red[2][i];
   }
-  if (tid < NV * 32) {
-    k_s[tid] = kx / sqrtf(tk + key_eps);
-    q_s[tid] = qx / sqrtf(tq + key_eps) * (1.0f / sqrtf((float)d));
+  const float ik = 1.0f / sqrtf(tk + key_eps), iq = 1.0f / (sqrtf(tq + key_eps) * sqrtf((float)d));
+  kq *= ik * iq;
+  if (tid < NV * RG) {
+    k_s[tid] = kx * ik;
+    q_s[tid] = qx * iq;
     w_s[tid] = wx;
   }
   __syncthreads();
-  // sums over the key channels of four columns: the thread's, its warp's, then all warps'
-  auto total = [&](float (&a)[4]) {
-#pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      a[j] += __shfl_xor_sync(0xffffffffu, a[j], 8);
-      a[j] += __shfl_xor_sync(0xffffffffu, a[j], 16);
-    }
-    if (lane < 8) *reinterpret_cast<float4*>(&part[warp][cq * 4]) = make_float4(a[0], a[1], a[2], a[3]);
-    __syncthreads();
-    a[0] = a[1] = a[2] = a[3] = 0.0f;
-#pragma unroll
-    for (int w = 0; w < ST_THREADS / 32; ++w) {
-      const float4 f = *reinterpret_cast<const float4*>(&part[w][cq * 4]);
-      a[0] += f.x; a[1] += f.y; a[2] += f.z; a[3] += f.w;
-    }
-  };
-  float a[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+  // a: S'^T k, o: S'^T q of four columns: the thread's key channels, its warp's, then all warps'
+  float a[4] = {0.0f, 0.0f, 0.0f, 0.0f}, o[4] = {0.0f, 0.0f, 0.0f, 0.0f};
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
-    const float w = w_s[rg + 32 * i], k = k_s[rg + 32 * i];
+    const float w = w_s[rg + RG * i], k = k_s[rg + RG * i], q = q_s[rg + RG * i];
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       S[i][j] *= w;
       a[j] = fmaf(k, S[i][j], a[j]);
-    }
-  }
-  total(a);
-  float u[4], o[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-#pragma unroll
-  for (int j = 0; j < 4; ++j) u[j] = beta * (v4[j] - a[j]);
-#pragma unroll
-  for (int i = 0; i < NV; ++i) {
-    const float k = k_s[rg + 32 * i], q = q_s[rg + 32 * i];
-#pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      S[i][j] = fmaf(k, u[j], S[i][j]);
       o[j] = fmaf(q, S[i][j], o[j]);
     }
-    const int c = rg + 32 * i;
-    if (c < d && col < dv) {
-      if (vec) {
-        *reinterpret_cast<float4*>(st + (size_t)c * dv + col) =
-            make_float4(S[i][0], S[i][1], S[i][2], S[i][3]);
-      } else {
-#pragma unroll
-        for (int j = 0; j < 4; ++j)
-          if (col + j < dv) st[(size_t)c * dv + col + j] = S[i][j];
-      }
-    }
   }
-  nb_launch_dependents();
-  __syncthreads();             // `part` is used again
-  total(o);
-  asm volatile("barrier.cluster.wait.aligned;\n" ::: "memory");
-  // the head's sum of squares: warp 0 has this CTA's columns, the cluster the rest
-  float mine = 0.0f;
+#pragma unroll
+  for (int m = CQ; m < 32; m <<= 1)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      a[j] += __shfl_xor_sync(0xffffffffu, a[j], m);
+      o[j] += __shfl_xor_sync(0xffffffffu, o[j], m);
+    }
+  if (lane < CQ) {
+    *reinterpret_cast<float4*>(&part[0][warp][cq * 4]) = make_float4(a[0], a[1], a[2], a[3]);
+    *reinterpret_cast<float4*>(&part[1][warp][cq * 4]) = make_float4(o[0], o[1], o[2], o[3]);
+  }
+  __syncthreads();
+  float u[4];
+  a[0] = a[1] = a[2] = a[3] = 0.0f;
+#pragma unroll
+  for (int w = 0; w < NW; ++w) {
+    const float4 f = *reinterpret_cast<const float4*>(&part[0][w][cq * 4]);
+    a[0] += f.x; a[1] += f.y; a[2] += f.z; a[3] += f.w;
+  }
+#pragma unroll
+  for (int j = 0; j < 4; ++j) u[j] = beta * (v4[j] - a[j]);
+  // warp 0 has the CTA's outputs: lane cq's four columns
+  float ss = 0.0f;
   if (warp == 0) {
-    // lane l takes column l: it sits in lane l / 4 (cq), number l % 4
-    const float x0 = __shfl_sync(0xffffffffu, o[0], lane >> 2), x1 = __shfl_sync(0xffffffffu, o[1], lane >> 2);
-    const float x2 = __shfl_sync(0xffffffffu, o[2], lane >> 2), x3 = __shfl_sync(0xffffffffu, o[3], lane >> 2);
-    const int j = lane & 3;
-    mine = j == 0 ? x0 : j == 1 ? x1 : j == 2 ? x2 : x3;
-    if (split * ST_COLS + lane >= dv) mine = 0.0f;
-    const float ss = nb_warp_sum(mine * mine);
-    if (lane < n_splits) {
+    o[0] = o[1] = o[2] = o[3] = 0.0f;
+#pragma unroll
+    for (int w = 0; w < NW; ++w) {
+      const float4 f = *reinterpret_cast<const float4*>(&part[1][w][cq * 4]);
+      o[0] += f.x; o[1] += f.y; o[2] += f.z; o[3] += f.w;
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      o[j] = fmaf(kq, u[j], o[j]);
+      if (tid < CQ && col + j < dv) ss = fmaf(o[j], o[j], ss);
+    }
+    ss = nb_warp_sum(ss);
+  }
+  if (n_splits > 1) {          // the head's sum of squares, over the cluster
+    asm volatile("barrier.cluster.wait.aligned;\n" ::: "memory");
+    if (warp == 0 && lane < n_splits) {
       const unsigned local = (unsigned)__cvta_generic_to_shared(&square[split]);
       unsigned remote;
       asm volatile("mapa.shared::cluster.u32 %0, %1, %2;\n" : "=r"(remote) : "r"(local), "r"(lane));
       asm volatile("st.shared::cluster.f32 [%0], %1;\n" ::"r"(remote), "f"(ss) : "memory");
     }
+    asm volatile("barrier.cluster.arrive.release.aligned;\n" ::: "memory");
   }
-  asm volatile("barrier.cluster.arrive.release.aligned;\n" ::: "memory");
-  asm volatile("barrier.cluster.wait.acquire.aligned;\n" ::: "memory");
-  if (warp == 0 && split * ST_COLS + lane < dv) {
-    float ss = 0.0f;
+  nb_launch_dependents();
+  // the state, while the squares travel
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = rg + RG * i;
+    if (c >= d || col >= dv) continue;
+    const float k = k_s[c];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) S[i][j] = fmaf(k, u[j], S[i][j]);
+    if (vec) {
+      *reinterpret_cast<float4*>(st + (size_t)c * dv + col) =
+          make_float4(S[i][0], S[i][1], S[i][2], S[i][3]);
+    } else {
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (col + j < dv) st[(size_t)c * dv + col + j] = S[i][j];
+    }
+  }
+  if (n_splits > 1) {
+    asm volatile("barrier.cluster.wait.acquire.aligned;\n" ::: "memory");
+    ss = 0.0f;
     for (int i = 0; i < n_splits; ++i) ss += square[i];
-    const int c = split * ST_COLS + lane;
-    out[(size_t)r * hv + h * dv + c] = nb_from_f32<TOut>(
-        mine * (1.0f / sqrtf(ss / (float)dv + eps)) * norm_w[c] * nb_sigmoid(gate));
+  }
+  if (tid < CQ) {
+    const float inv = 1.0f / sqrtf(ss / (float)dv + eps);
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+      if (col + j < dv)
+        out[(size_t)r * hv + h * dv + col + j] =
+            nb_from_f32<TOut>(o[j] * inv * norm_w[col + j] * nb_sigmoid(gate[j]));
   }
 }
 
@@ -935,21 +954,28 @@ NB_EXPORT int nb_gated_delta_step(const float* qkv, int qkv_stride, const float*
   const Source src{qkv, qkv_stride, 0, nullptr, 0, nullptr, 0, 2 * n_kv_heads * d + n_heads * dv, beta,
                    beta_stride, beta_col, low, low_stride, decay_col, gate_col, a_log, dt_bias};
   const int vec = dv % 4 == 0 && state_stride % 4 == 0 && (uintptr_t)state % 16 == 0;
-  const int splits = (dv + ST_COLS - 1) / ST_COLS;
+  // a CTA per 128 columns where that fills the GPU (and the state of a head fits its registers);
+  // measured at 64 sequences of 16 heads of 128: 48 us with the convolution, 66 with 32 columns a CTA
+  const bool wide = d <= 128 && dv > 32 && (long long)n_heads * n_seqs * ((dv + 127) / 128) >= 2 * 148;
+  const int cols = wide ? 128 : 32, splits = (dv + cols - 1) / cols;
   const dim3 grid(splits, n_heads, n_seqs);
-#define NB_GS(NV, TO)                                                                             \
-  NB_CUDA(nb_launch_clusters(gated_delta_step_kernel<NV, TO>, grid, dim3(ST_THREADS), 0, stream,  \
-                             splits, src, key_eps, norm_w, eps, cu_rows, seq_slot, state,         \
+#define NB_GS(NV, COLS, TO)                                                                       \
+  NB_CUDA(nb_launch_clusters(gated_delta_step_kernel<NV, COLS, TO>, grid, dim3(ST_THREADS), 0,    \
+                             stream, splits, src, key_eps, norm_w, eps, cu_rows, seq_slot, state, \
                              state_stride, (TO*)out, n_heads, n_kv_heads, d, dv, vec))
-#define NB_GS_T(NV)                                                                               \
+#define NB_GS_T(NV, COLS)                                                                         \
   do {                                                                                            \
-    if (out_dtype == NB_F32) NB_GS(NV, float);                                                    \
-    else NB_GS(NV, __nv_bfloat16);                                                                \
+    if (out_dtype == NB_F32) NB_GS(NV, COLS, float);                                              \
+    else NB_GS(NV, COLS, __nv_bfloat16);                                                          \
   } while (0)
-  if (d <= 32) NB_GS_T(1);
-  else if (d <= 64) NB_GS_T(2);
-  else if (d <= 128) NB_GS_T(4);
-  else NB_GS_T(8);
+  if (wide) {
+    if (d <= 32) NB_GS_T(4, 128);
+    else if (d <= 64) NB_GS_T(8, 128);
+    else NB_GS_T(16, 128);
+  } else if (d <= 32) NB_GS_T(1, 32);
+  else if (d <= 64) NB_GS_T(2, 32);
+  else if (d <= 128) NB_GS_T(4, 32);
+  else NB_GS_T(8, 32);
 #undef NB_GS_T
 #undef NB_GS
   NB_CHECK_LAUNCH("gated_delta_step");

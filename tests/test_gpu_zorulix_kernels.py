@@ -350,7 +350,7 @@ RECURRENCES = [(1, 1, 1, 1), (2, 1, 3, 5), (4, 2, 9, 13), (3, 3, 32, 32), (2, 2,
 
 @pytest.mark.parametrize("H,G,d,dv", RECURRENCES)
 def test_the_recurrence_whole_in_portions_and_token_by_token(ops, H, G, d, dv):
-    """However the sequence is cut (blocks of four tokens start anywhere), outputs and state."""
+    """However the sequence is cut (blocks of eight tokens start anywhere), outputs and state."""
     T, eps = 75, 1e-5
     rows, weights = _recurrence_inputs(T, H, G, d, dv, 7), _weights(H, d, dv)
     ref, S = _plain_recurrence(*rows, *weights, H, G, d, dv, eps)
@@ -448,6 +448,24 @@ def test_unequal_sequences_in_one_batch(ops, dtype, H, G, d, dv):
                 assert float(got[i].abs().max()) == 0.0 and torch.equal(state[slots[2]], before)
             else:
                 _close(got[i], refs[i][n + step], TOL[dtype], f"{n} tokens and {step + 1}")
+
+
+@pytest.mark.parametrize("H,G,d,dv", [(16, 16, 128, 128), (16, 8, 64, 96), (12, 4, 30, 130), (16, 2, 20, 33)])
+def test_one_token_steps_of_many_heads(ops, H, G, d, dv):
+    """Enough heads that a CTA takes all or 128 of a head's columns: twenty-four sequences, three
+    tokens one by one, against each alone."""
+    n, T, eps = 24, 3, 1e-5
+    weights = _weights(H, d, dv)
+    data = [_recurrence_inputs(T, H, G, d, dv, 5 * i) for i in range(n)]
+    refs = [_plain_recurrence(*x, *weights, H, G, d, dv, eps) for x in data]
+    state = torch.zeros(n, H * d * dv, device=DEV)
+    slots = [(7 * i) % n for i in range(n)]
+    for t in range(T):
+        lay = build_layout([(s, [1], []) for s in slots], [t] * n, torch.device(DEV))
+        rows = [torch.stack([x[j][t] for x in data]) for j in range(3)]
+        got = _run(ops, "float32", rows, weights, lay, state, H, G, d, dv, eps)
+        _close(got, torch.stack([ref[t] for ref, _ in refs]), 5e-5, f"token {t}")
+    _close(state[slots].view(n, H, d, dv), torch.stack([S for _, S in refs]), 2e-5, "state")
 
 
 @pytest.mark.parametrize("H,G,d,dv", [(2, 1, 12, 10), (2, 2, 12, 10), (3, 3, 64, 64), (2, 2, 128, 128),
