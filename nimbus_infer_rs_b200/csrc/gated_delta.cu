@@ -648,7 +648,7 @@ gated_delta_walk_kernel(const float* records, const int* cu_rows, const int* seq
 constexpr int ST_THREADS = 256;
 
 template <int NV, int COLS, typename TOut>
-__global__ void __launch_bounds__(ST_THREADS, COLS == 128 ? 2 : 1)
+__global__ void __launch_bounds__(ST_THREADS, COLS == 128 ? 2 : (NV > 4 ? 1 : 4))
 gated_delta_step_kernel(Source src, float key_eps, const float* __restrict__ norm_w, float eps,
                         const int* cu_rows, const int* seq_slot, float* state, int state_stride,
                         TOut* out, int n_heads, int n_kv_heads, int d, int dv, int vec) {

@@ -1121,7 +1121,7 @@ class CudaBackend:
                        st.stride(0), _ptr(out), dtype_code(out.dtype), H, G, d, dv, layout.n_seqs,
                        self._stream())
             return
-        # what every block of four tokens does to the state, and the outputs before their norm
+        # what every block of eight tokens does to the state, and the outputs before their norm
         records = torch.empty(self.lib.nb_gated_delta_scratch(n, layout.n_seqs, H, d, dv),
                               device=out.device, dtype=torch.float32)
         o_raw = torch.empty((n, H * dv), device=out.device, dtype=torch.float32)
